@@ -10,7 +10,8 @@ A model is described as data:
 * ``PlanEntry`` - one execution of a layer.  The plan is the order in which layers run; it may name
   a layer twice (each run that writes has a cache of its own) or let a run read the cache that an
   earlier run wrote (``reads_cache_of``), in which case it writes nothing.  An entry with
-  ``adds_embedding`` starts a new pass over looped layers: the embedding rows join the stream again.
+  ``adds_embedding`` starts a new pass over looped layers: the embedding rows join the stream again;
+  with ``adds_vector`` it is one learned vector, the same for every token.
 
 The reference builds one fixed stack (src/models/llama.py:112-124) and loops over it
 (:183-189); it has no layer specs and no plan.
@@ -71,6 +72,9 @@ class PlanEntry:
     # the embedding rows (the stream as it was before the first entry) are added to the stream
     # before this entry runs
     adds_embedding: bool = False
+    # this row of the model's plan vectors (``ModelConfig.plan_vectors``) is added to every row of
+    # the stream before this entry runs
+    adds_vector: "int | None" = None
 
 
 @dataclass(frozen=True)
@@ -105,6 +109,11 @@ class ModelConfig:
         """A norm on the embedding rows before the first layer (its tensor under the prefix
         ``tensor_names()["embedding_norm"]``), or None."""
         return None
+
+    def plan_vectors(self) -> int:
+        """How many vectors [width] the plan's entries name with ``adds_vector`` (one tensor
+        [count, width] called ``tensor_names()["plan_vectors"]``); 0: none, and no tensor."""
+        return 0
 
     @property
     def logit_softcap(self) -> "float | None":

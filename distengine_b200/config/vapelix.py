@@ -59,7 +59,8 @@ def _rotation(m: Mapping[str, Any], where: str, rot_dim: int) -> tuple:
     return base, scaling
 
 
-def _latent_attention(m: Mapping[str, Any], where: str) -> dict:
+def latent_attention_keys(m: Mapping[str, Any], where: str) -> dict:
+    """The sizes and constants of a latent-attention mixer's section."""
     rot_dim = m.get("rot_dim")
     if type(rot_dim) is not int or rot_dim < 0 or rot_dim % 2:
         raise ConfigError(f"config.json: '{where}rot_dim' ({rot_dim!r}) must be an even number "
@@ -93,9 +94,10 @@ def _feed_forward(mlp: Any, where: str) -> "dict | None":
                       f"'moe'")
 
 
-def _freeze(value):
+def freeze(value):
+    """Nested dictionaries as sorted tuples of pairs, which a frozen configuration can hold."""
     if isinstance(value, dict):
-        return tuple(sorted((k, _freeze(v)) for k, v in value.items()))
+        return tuple(sorted((k, freeze(v)) for k, v in value.items()))
     return value
 
 
@@ -130,8 +132,8 @@ class VapelixConfig(ModelConfig):
             if entry.get("type") != "latent_attention":
                 raise ConfigError(f"config.json: '{where}type' is {entry.get('type')!r}; this "
                                   f"design has 'latent_attention'")
-            mixer = _latent_attention(_section(entry, "mixer", where), where + "mixer.")
-            layers.append((_freeze(mixer), _freeze(_feed_forward(entry.get("mlp"), where))))
+            mixer = latent_attention_keys(_section(entry, "mixer", where), where + "mixer.")
+            layers.append((freeze(mixer), freeze(_feed_forward(entry.get("mlp"), where))))
         loop = None
         if data.get("loop") is not None:
             section = _section(data, "loop", "")

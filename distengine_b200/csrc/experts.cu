@@ -15,6 +15,16 @@
 // weight * h for them).  An expert's up product may have no activation (kind 5), for experts whose
 // gate and up rows are stacked and joined by a kernel after the product.
 //
+// A third (`mode` 2): s = sigmoid(z); the choice scores are s + bias; the experts form `groups`
+// equal groups of neighbours whose value is the sum of their two largest choice scores, only
+// experts of the `keep` best groups can be chosen (ties: the lower group); the weights are the
+// chosen s over their sum (+ 1e-20), times `scale`.  With `side`, the router has one row more than
+// there are outputs: side[n] = sigmoid of it, a token's factor on a shared expert, whose rows
+// `combine` then adds.
+//
+// clipped_glu is a join of gate and up with limits: g sigmoid(sharpness g) (u + 1) with
+// g = min(gate, limit), u = up clamped to +- limit.
+//
 // Every output element is one chain of multiply-adds over its inputs in ascending order, and a
 // token's result does not depend on which tokens share its tile, its expert or its step.  The
 // number of tiles that are launched depends on the number of tokens only (tiles without an expert
@@ -35,14 +45,36 @@ constexpr int MAX_TOP = 32;
 // token's logits do not depend on its step.  Then warp 0 picks the `top` largest (ties: the lower
 // index) and forms the softmax over them.  Shared memory: [9][experts] floats.
 constexpr int ROUTE_WARPS = 8;
+
+// The index of the largest of z[0 .. count) (ties: the lower index) and its value, by one warp.
+__device__ __forceinline__ int warp_arg_max(const float* z, int count, int lane, float& value) {
+    float v = -INFINITY;
+    int at = 0x7fffffff;
+    for (int e = lane; e < count; e += 32) {
+        const float c = z[e];
+        if (c > v || (c == v && e < at)) { v = c; at = e; }
+    }
+    if (at == 0x7fffffff) v = -INFINITY;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+        if (ov > v || (ov == v && oa < at)) { v = ov; at = oa; }
+    }
+    value = v;
+    return at < count ? at : 0;                      // (numbers that compare with nothing)
+}
+
 template <typename T>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 route_kernel(const T* __restrict__ h, int ldh, const float* __restrict__ w,
-             const float* __restrict__ bias, int n, int width, int experts, int top, int mode,
-             int* __restrict__ chosen, float* __restrict__ weight) {
+             const float* __restrict__ bias, int n, int width, int outputs, int top, int mode,
+             int groups, int keep, float scale, int* __restrict__ chosen,
+             float* __restrict__ weight, float* __restrict__ side) {
     extern __shared__ float zs[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int row = blockIdx.x;
+    const int experts = outputs + (side != nullptr ? 1 : 0);      // rows of the router
     float* z = zs + (size_t)ROUTE_WARPS * experts;
     pdl_wait();
     pdl_trigger();
@@ -80,41 +112,66 @@ route_kernel(const T* __restrict__ h, int ldh, const float* __restrict__ w,
         float t = 0.0f;
 #pragma unroll
         for (int k = 0; k < ROUTE_WARPS; ++k) t += zs[(size_t)k * experts + e];
-        z[e] = mode == 1 ? t : t + bias[e];
+        z[e] = mode != 0 || e >= outputs ? t : t + bias[e];
     }
     __syncthreads();
     if (warp != 0) return;
+    if (side != nullptr && lane == 0) side[row] = 1.0f / (1.0f + expf(-z[outputs]));
     float best[MAX_TOP];
     float total = 0.0f;
     if (mode == 1) {
         // scores over all outputs; z becomes score + correction, the scores stay in zs
         float top_z = -INFINITY;
-        for (int e = lane; e < experts; e += 32) top_z = fmaxf(top_z, z[e]);
+        for (int e = lane; e < outputs; e += 32) top_z = fmaxf(top_z, z[e]);
         top_z = warp_max(top_z);
         float sum = 0.0f;
-        for (int e = lane; e < experts; e += 32) sum += expf(z[e] - top_z);
+        for (int e = lane; e < outputs; e += 32) sum += expf(z[e] - top_z);
         sum = warp_sum(sum);
-        for (int e = lane; e < experts; e += 32) {
+        for (int e = lane; e < outputs; e += 32) {
             const float sc = expf(z[e] - top_z) / sum;
             zs[e] = sc;
             z[e] = sc + bias[e];
         }
         __syncwarp();
+    } else if (mode == 2) {
+        for (int e = lane; e < outputs; e += 32) {
+            const float sc = 1.0f / (1.0f + expf(-z[e]));
+            zs[e] = sc;
+            z[e] = sc + bias[e];
+        }
+        __syncwarp();
+        if (keep < groups) {
+            float* value = zs + outputs;                 // [groups], then [groups] kept or not
+            float* open = value + groups;
+            const int size = outputs / groups;
+            for (int g = lane; g < groups; g += 32) {
+                float first = -INFINITY, second = -INFINITY;
+                for (int e = g * size; e < (g + 1) * size; ++e) {
+                    const float c = z[e];
+                    if (c > first) { second = first; first = c; }
+                    else if (c > second) second = c;
+                }
+                value[g] = size > 1 ? first + second : first;
+                open[g] = 0.0f;
+            }
+            __syncwarp();
+            for (int k = 0; k < keep; ++k) {
+                float v;
+                const int at = warp_arg_max(value, groups, lane, v);
+                if (lane == 0) {
+                    open[at] = 1.0f;
+                    value[at] = -INFINITY;
+                }
+                __syncwarp();
+            }
+            for (int e = lane; e < outputs; e += 32)
+                if (open[e / size] == 0.0f) z[e] = -INFINITY;
+            __syncwarp();
+        }
     }
     for (int k = 0; k < top; ++k) {
-        float v = -INFINITY;
-        int at = 0x7fffffff;
-        for (int e = lane; e < experts; e += 32) {
-            const float c = z[e];
-            if (c > v || (c == v && e < at)) { v = c; at = e; }
-        }
-        if (at == 0x7fffffff) v = -INFINITY;
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-            const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-            if (ov > v || (ov == v && oa < at)) { v = ov; at = oa; }
-        }
+        float v;
+        const int at = warp_arg_max(z, outputs, lane, v);
         best[k] = v;
         if (lane == 0) {
             chosen[(size_t)row * top + k] = at;
@@ -126,6 +183,16 @@ route_kernel(const T* __restrict__ h, int ldh, const float* __restrict__ w,
         if (lane == 0)
             for (int k = 0; k < top; ++k)
                 weight[(size_t)row * top + k] = zs[chosen[(size_t)row * top + k]];
+        return;
+    }
+    if (mode == 2) {
+        if (lane == 0) {
+            float sum = 0.0f;
+            for (int k = 0; k < top; ++k) sum += zs[chosen[(size_t)row * top + k]];
+            const float factor = scale / (sum + 1e-20f);
+            for (int k = 0; k < top; ++k)
+                weight[(size_t)row * top + k] = zs[chosen[(size_t)row * top + k]] * factor;
+        }
         return;
     }
     for (int k = 0; k < top; ++k) total += expf(best[k] - best[0]);
@@ -268,12 +335,14 @@ __global__ void gather_kernel(const T* __restrict__ h, int ldh, const int* __res
 }
 
 // chosen / experts / h: a pair whose choice is not below `experts` adds weight * h[n] (an expert
-// that hands its input on); chosen null: every pair has a row of y.
+// that hands its input on); chosen null: every pair has a row of y.  shared / side: side[n] *
+// shared[n] joins the sum (an expert that every token uses).
 template <typename T>
 __global__ void combine_kernel(const T* __restrict__ y, const float* __restrict__ weight, int top,
                                int width, size_t total, float* __restrict__ out,
                                const int* __restrict__ chosen, int experts,
-                               const T* __restrict__ h, int ldh) {
+                               const T* __restrict__ h, int ldh, const T* __restrict__ shared,
+                               const float* __restrict__ side) {
     pdl_wait();
     pdl_trigger();
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
@@ -287,7 +356,46 @@ __global__ void combine_kernel(const T* __restrict__ y, const float* __restrict_
                                      : to_float(y[(n * top + k) * width + i]);
             s = fmaf(weight[n * top + k], v, s);
         }
+        if (shared != nullptr) s = fmaf(side[n], to_float(shared[idx]), s);
         out[idx] = s;
+    }
+}
+
+__device__ __forceinline__ float clipped_gate(float gate, float up, float limit, float sharpness) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.0f + expf(-sharpness * g)) * (u + 1.0f);
+}
+
+// out[n, i] = clipped_gate(x[n, i], x[n, inner + i]); VEC: four outputs a thread and turn.
+template <typename T, int VEC>
+__global__ void clipped_glu_kernel(const T* __restrict__ x, int ldx, T* __restrict__ out, int ldo,
+                                   int inner, size_t total, float limit, float sharpness) {
+    pdl_wait();
+    pdl_trigger();
+    const int pieces = inner / VEC;
+    for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
+         idx += (size_t)gridDim.x * blockDim.x) {
+        const size_t n = idx / pieces;
+        const int i = VEC * (int)(idx - n * pieces);
+        if constexpr (VEC == 4) {
+            float g[4], u[4];
+            rows_product::load4<T>(x + n * ldx + i, 0, 4, true, g);
+            rows_product::load4<T>(x + n * ldx + inner + i, 0, 4, true, u);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) g[e] = clipped_gate(g[e], u[e], limit, sharpness);
+            if constexpr (sizeof(T) == 4) {
+                *reinterpret_cast<float4*>(out + n * ldo + i) = make_float4(g[0], g[1], g[2], g[3]);
+            } else {
+                const __nv_bfloat162 a = __floats2bfloat162_rn(g[0], g[1]);
+                const __nv_bfloat162 b = __floats2bfloat162_rn(g[2], g[3]);
+                *reinterpret_cast<uint2*>(out + n * ldo + i) =
+                    make_uint2(*reinterpret_cast<const unsigned*>(&a),
+                               *reinterpret_cast<const unsigned*>(&b));
+            }
+        } else {
+            out[n * ldo + i] = from_float<T>(clipped_gate(
+                to_float(x[n * ldx + i]), to_float(x[n * ldx + inner + i]), limit, sharpness));
+        }
     }
 }
 
@@ -302,19 +410,23 @@ DE_EXPORT int de_experts_tiles(int n, int top, int experts, int seg) {
 
 DE_EXPORT int de_experts_route(int dtype, const void* h, int ldh, const float* w,
                                const float* bias, int n, int width, int experts, int top,
-                               int mode, int* chosen, float* weight, void* stream) {
+                               int mode, int groups, int keep, float scale, int* chosen,
+                               float* weight, float* side, void* stream) {
     if (n <= 0) return 0;
     if (top <= 0 || top > MAX_TOP || top > experts || experts > 1024) return -2;
+    if (mode < 0 || mode > 2 || (mode == 2 && (groups <= 0 || experts % groups || keep <= 0 ||
+                                               keep > groups || top > experts / groups * keep)))
+        return -2;
     cudaStream_t s = (cudaStream_t)stream;
     const int warps = ROUTE_WARPS;
-    const size_t smem = (size_t)(warps + 1) * experts * sizeof(float);
+    const size_t smem = (size_t)(warps + 1) * (experts + (side != nullptr ? 1 : 0)) * sizeof(float);
     const dim3 grid(n);
     if (dtype == DE_BF16)
         return de_launch(route_kernel<__nv_bfloat16>, grid, dim3(warps * 32), smem, s,
                          (const __nv_bfloat16*)h, ldh, w, bias, n, width, experts, top, mode,
-                         chosen, weight);
+                         groups, keep, scale, chosen, weight, side);
     return de_launch(route_kernel<float>, grid, dim3(warps * 32), smem, s, (const float*)h, ldh, w,
-                     bias, n, width, experts, top, mode, chosen, weight);
+                     bias, n, width, experts, top, mode, groups, keep, scale, chosen, weight, side);
 }
 
 DE_EXPORT int de_experts_group(const int* chosen, int pairs, int experts, int tiles, int seg,
@@ -380,7 +492,8 @@ DE_EXPORT int de_experts_down(int dtype, const void* inner, const void* down, co
 
 DE_EXPORT int de_experts_combine(int dtype, const void* y, const float* weight, int n, int top,
                                  int width, float* out, const int* chosen, int experts,
-                                 const void* h, int ldh, void* stream) {
+                                 const void* h, int ldh, const void* shared, const float* side,
+                                 void* stream) {
     if (n <= 0) return 0;
     const size_t total = (size_t)n * width;
     size_t blocks = (total + 255) / 256;
@@ -389,8 +502,29 @@ DE_EXPORT int de_experts_combine(int dtype, const void* y, const float* weight, 
     if (dtype == DE_BF16)
         return de_launch(combine_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(256), 0, s,
                          (const __nv_bfloat16*)y, weight, top, width, total, out, chosen, experts,
-                         (const __nv_bfloat16*)h, ldh);
+                         (const __nv_bfloat16*)h, ldh, (const __nv_bfloat16*)shared, side);
     return de_launch(combine_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, s,
                      (const float*)y, weight, top, width, total, out, chosen, experts,
-                     (const float*)h, ldh);
+                     (const float*)h, ldh, (const float*)shared, side);
+}
+
+DE_EXPORT int de_clipped_glu(int dtype, const void* x, int ldx, void* out, int ldo, int n,
+                             int inner, float limit, float sharpness, void* stream) {
+    if (n <= 0 || inner <= 0) return 0;
+    cudaStream_t s = (cudaStream_t)stream;
+    const bool vec = inner % 4 == 0 && ldx % 4 == 0 && ldo % 4 == 0 && (uintptr_t)x % 16 == 0 &&
+                     (uintptr_t)out % 16 == 0;
+    const size_t total = vec ? (size_t)n * (inner / 4) : (size_t)n * inner;
+    size_t blocks = (total + 255) / 256;
+    if (blocks > 148 * 32) blocks = 148 * 32;
+#define GLU(T, V)                                                                               \
+    return de_launch(clipped_glu_kernel<T, V>, dim3((unsigned)blocks), dim3(256), 0, s,         \
+                     (const T*)x, ldx, (T*)out, ldo, inner, total, limit, sharpness)
+    if (dtype == DE_BF16) {
+        if (vec) GLU(__nv_bfloat16, 4);
+        GLU(__nv_bfloat16, 1);
+    }
+    if (vec) GLU(float, 4);
+    GLU(float, 1);
+#undef GLU
 }

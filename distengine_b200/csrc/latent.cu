@@ -21,15 +21,16 @@ DE_DEFINE_PDL_SWITCH
 namespace {
 
 // One block a token.  kv row = [c raw (rank) | key part (rot)], q row = H heads of [plain (dim) |
-// rotated part (rot)]; qa row = H heads of [.. (rank, written by heads_product) | rotated (rot)].
+// rotated part (rot)]; the pairs of a rotated part are (i, i + rot / 2), or with `adjacent`
+// (2i, 2i + 1); qa row = H heads of [.. (rank, written by heads_product) | rotated (rot)].
 template <typename T, typename W>
 __global__ void latent_write_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ kv,
                                     int ldkv, T* __restrict__ qa, int ldqa,
                                     const int* __restrict__ positions,
                                     const int* __restrict__ token_slot,
                                     const double* __restrict__ freq, float magnitude,
-                                    const W* __restrict__ norm_w, float eps, int H, int dim,
-                                    int rot, int rank, T* __restrict__ pages,
+                                    const W* __restrict__ norm_w, float eps, int adjacent, int H,
+                                    int dim, int rot, int rank, T* __restrict__ pages,
                                     const int* __restrict__ block_table, int table_stride,
                                     int page, int num_pages, int* __restrict__ status) {
     extern __shared__ float cs[];                    // [rot]: cosines, then sines, of the position
@@ -58,12 +59,13 @@ __global__ void latent_write_kernel(const T* __restrict__ q, int ldq, const T* _
     T* qar = qa + (size_t)n * ldqa;
     for (int e = threadIdx.x; e < H * half; e += blockDim.x) {
         const int h = e / half, i = e - h * half;
-        const float a = to_float(qr[h * (dim + rot) + dim + i]);
-        const float b = to_float(qr[h * (dim + rot) + dim + half + i]);
+        const int ia = adjacent ? 2 * i : i, ib = adjacent ? 2 * i + 1 : half + i;
+        const float a = to_float(qr[h * (dim + rot) + dim + ia]);
+        const float b = to_float(qr[h * (dim + rot) + dim + ib]);
         float ra, rb;
         rope_rotate(a, b, cs[i], cs[half + i], ra, rb);
-        qar[h * row_dim + rank + i] = from_float<T>(ra);
-        qar[h * row_dim + rank + half + i] = from_float<T>(rb);
+        qar[h * row_dim + rank + ia] = from_float<T>(ra);
+        qar[h * row_dim + rank + ib] = from_float<T>(rb);
     }
     if (page_id < 0 || page_id >= num_pages) {       // never written outside the pool
         if (threadIdx.x == 0) atomicExch(status, 1);
@@ -75,11 +77,12 @@ __global__ void latent_write_kernel(const T* __restrict__ q, int ldq, const T* _
         dst[i] = from_float<T>(v * to_float(norm_w[i]));
     }
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        const int ia = adjacent ? 2 * i : i, ib = adjacent ? 2 * i + 1 : half + i;
         float ra, rb;
-        rope_rotate(to_float(kvr[rank + i]), to_float(kvr[rank + half + i]), cs[i], cs[half + i],
-                    ra, rb);
-        dst[rank + i] = from_float<T>(ra);
-        dst[rank + half + i] = from_float<T>(rb);
+        rope_rotate(to_float(kvr[rank + ia]), to_float(kvr[rank + ib]), cs[i], cs[half + i], ra,
+                    rb);
+        dst[rank + ia] = from_float<T>(ra);
+        dst[rank + ib] = from_float<T>(rb);
     }
 }
 
@@ -126,8 +129,8 @@ heads_product_kernel(const TA* __restrict__ a, int lda, int lda_h, const TW* __r
 DE_EXPORT int de_latent_write(int dtype, int weight_dtype, const void* q, int ldq, const void* kv,
                               int ldkv, void* qa, int ldqa, const int* positions,
                               const int* token_slot, const double* freq, float magnitude,
-                              const void* norm_w, float eps, int H, int dim, int rot, int rank,
-                              void* pages, const int* block_table, int table_stride, int page,
+                              const void* norm_w, float eps, int adjacent, int H, int dim,
+                              int rot, int rank, void* pages, const int* block_table, int table_stride, int page,
                               int num_pages, int n, int* status, void* stream) {
     if (n <= 0) return 0;
     if (rot < 0 || rot % 2 || rank <= 0 || dim <= 0 || H <= 0) return -2;
@@ -136,7 +139,7 @@ DE_EXPORT int de_latent_write(int dtype, int weight_dtype, const void* q, int ld
 #define LW(T, W)                                                                                \
     return de_launch(latent_write_kernel<T, W>, dim3(n), dim3(128), smem, s, (const T*)q, ldq,   \
                      (const T*)kv, ldkv, (T*)qa, ldqa, positions, token_slot, freq, magnitude,  \
-                     (const W*)norm_w, eps, H, dim, rot, rank, (T*)pages, block_table,          \
+                     (const W*)norm_w, eps, adjacent, H, dim, rot, rank, (T*)pages, block_table,          \
                      table_stride, page, num_pages, status)
     if (dtype == DE_BF16) {
         if (weight_dtype == DE_BF16) LW(__nv_bfloat16, __nv_bfloat16);

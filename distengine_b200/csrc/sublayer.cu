@@ -9,6 +9,9 @@
 //                      layer's result so far, c a learned vector of the layer)
 //   poly_norm          out = a N(z) + b N(z^2) + c N(z^3) + e, N dividing a row by its root mean
 //                      square (eps inside the root), powers element by element
+//   join_rmsnorm       x <- x + y / sqrt(mean(y^2) + eps) * w (+ v) and out = the RMS norm of the
+//                      new x: the norm on a branch's result, the sum (with a vector v that every
+//                      row receives) and the norm before the next branch in one pass
 //
 // All sums, statistics and the stream are float32 whatever the activation type; every kernel that
 // writes the stream can also write its rounding to the activation type, which the next matrix
@@ -118,6 +121,23 @@ template <> struct Chunk<__nv_bfloat16> {
     }
 };
 
+// four neighbouring elements, 8 or 16 bytes
+__device__ __forceinline__ void load4(const float* p, float (&f)[4]) { Chunk<float>::load(p, f); }
+__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&f)[4]) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    f[0] = __uint_as_float(u.x << 16);
+    f[1] = __uint_as_float(u.x & 0xffff0000u);
+    f[2] = __uint_as_float(u.y << 16);
+    f[3] = __uint_as_float(u.y & 0xffff0000u);
+}
+__device__ __forceinline__ void store4(float* p, const float (&f)[4]) { Chunk<float>::store(p, f); }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&f)[4]) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]);
+    const __nv_bfloat162 b = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&a),
+                                              *reinterpret_cast<const unsigned*>(&b));
+}
+
 // Three sums over a block at once; every thread gets the results.  The order of the additions
 // depends on the block's size only.
 __device__ __forceinline__ void block_sum3(float& a, float& b, float& c, float* scratch /* 99 */) {
@@ -197,6 +217,104 @@ __global__ void poly_norm_kernel(const T* __restrict__ z, int ldz, const float* 
             const float v = to_float(zr[i]), v2 = v * v;
             out[row * ldo + i] = from_float<T>(v * i1 + v2 * i2 + v2 * v * i3 + e0);
         }
+    }
+}
+
+// Y: the branch's type; T: the output's; W: of both norm weights.  y null: no branch.  wy null: the
+// branch joins as it is.  vec null: no vector.  out null: the sum only.  rows: out[i] is the norm
+// of row rows[i], and x stays as it is.  A thread holds CHUNKS groups of four neighbouring elements
+// of the row in registers (CHUNKS 0: the row lies in shared memory, any width).
+struct Join {
+    const void *wy, *w;
+    const float* vec;
+    const int* rows;
+    int width;
+    float eps_y, eps;
+};
+
+template <typename T, typename Y, typename W, int CHUNKS>
+__global__ void join_rmsnorm_kernel(float* __restrict__ x, const Y* __restrict__ y,
+                                    T* __restrict__ out, Join j) {
+    __shared__ float scratch[33];
+    const int row = j.rows ? j.rows[blockIdx.x] : (int)blockIdx.x;
+    float* xr = x + (size_t)row * j.width;
+    const Y* yr = y ? y + (size_t)row * j.width : nullptr;
+    const W *wy = (const W*)j.wy, *w = (const W*)j.w;
+    T* o = out ? out + (size_t)blockIdx.x * j.width : nullptr;
+    pdl_wait();
+    if constexpr (CHUNKS > 0) {
+        const int quads = j.width >> 2;
+        float v[CHUNKS][4], b[CHUNKS][4];
+        float ss = 0.0f;
+#pragma unroll
+        for (int c = 0; c < CHUNKS; ++c) {
+            const int q = threadIdx.x + c * blockDim.x;
+            if (q < quads) {
+                load4(xr + 4 * q, v[c]);
+                if (yr) load4(yr + 4 * q, b[c]);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    if (!yr) b[c][e] = 0.0f;
+                    ss = fmaf(b[c][e], b[c][e], ss);
+                }
+            }
+        }
+        float inv = 1.0f;
+        if (wy) inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)j.width + j.eps_y);
+        ss = 0.0f;
+#pragma unroll
+        for (int c = 0; c < CHUNKS; ++c) {
+            const int q = threadIdx.x + c * blockDim.x;
+            if (q < quads) {
+                float g[4] = {1.0f, 1.0f, 1.0f, 1.0f}, a[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+                if (wy) load4(wy + 4 * q, g);
+                if (j.vec) load4(j.vec + 4 * q, a);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    v[c][e] = v[c][e] + b[c][e] * inv * g[e] + a[e];
+                    ss = fmaf(v[c][e], v[c][e], ss);
+                }
+                if (!j.rows) store4(xr + 4 * q, v[c]);
+            }
+        }
+        if (!o) return;
+        inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)j.width + j.eps);
+        pdl_trigger();
+#pragma unroll
+        for (int c = 0; c < CHUNKS; ++c) {
+            const int q = threadIdx.x + c * blockDim.x;
+            if (q < quads) {
+                float g[4];
+                load4(w + 4 * q, g);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) g[e] = v[c][e] * inv * g[e];
+                store4(o + 4 * q, g);
+            }
+        }
+    } else {
+        extern __shared__ float held[];              // [width]
+        float inv = 1.0f, ss = 0.0f;
+        if (wy) {
+            for (int i = threadIdx.x; i < j.width; i += blockDim.x) {
+                const float b = yr ? to_float(yr[i]) : 0.0f;
+                ss = fmaf(b, b, ss);
+            }
+            inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)j.width + j.eps_y);
+        }
+        ss = 0.0f;
+        for (int i = threadIdx.x; i < j.width; i += blockDim.x) {
+            const float b = yr ? to_float(yr[i]) : 0.0f;
+            const float v = xr[i] + b * inv * (wy ? to_float(wy[i]) : 1.0f) +
+                            (j.vec ? j.vec[i] : 0.0f);
+            held[i] = v;
+            ss = fmaf(v, v, ss);
+            if (!j.rows) xr[i] = v;
+        }
+        if (!o) return;
+        inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)j.width + j.eps);
+        pdl_trigger();
+        for (int i = threadIdx.x; i < j.width; i += blockDim.x)
+            o[i] = from_float<T>(held[i] * inv * to_float(w[i]));
     }
 }
 
@@ -288,4 +406,51 @@ DE_EXPORT int de_poly_norm(int dtype, const void* z, int ldz, const float* coef,
     if (vec) POLY(float, true);
     POLY(float, false);
 #undef POLY
+}
+
+// dtype: of out; y_dtype: of y; weight_dtype: of both weights.  n_out: rows of x, or of `rows`.
+DE_EXPORT int de_join_rmsnorm(int dtype, int y_dtype, int weight_dtype, float* x, const void* y,
+                              const void* wy, float eps_y, const float* vec, const void* w,
+                              float eps, void* out, const int* rows, int n_out, int width,
+                              void* stream) {
+    if (n_out <= 0) return 0;
+    if (dtype == DE_F32 && y_dtype != DE_F32) return -2;
+    cudaStream_t s = (cudaStream_t)stream;
+    const Join j = {wy, w, vec, rows, width, eps_y, eps};
+    const bool aligned = width % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0 &&
+                         (uintptr_t)wy % 16 == 0 && (uintptr_t)vec % 16 == 0 &&
+                         (uintptr_t)w % 16 == 0 && (uintptr_t)out % 16 == 0;
+    const int quads = width / 4;
+    const size_t smem = (size_t)width * sizeof(float);
+    if (smem > 200 * 1024) return -2;
+#define JOIN_AS(T, Y, W, CH, TH, SM)                                                             \
+    return de_launch(join_rmsnorm_kernel<T, Y, W, CH>, dim3(n_out), dim3(TH), SM, s, x,          \
+                     (const Y*)y, (T*)out, j)
+#define JOIN(T, Y, W)                                                                            \
+    do {                                                                                         \
+        if (aligned && quads <= 128) JOIN_AS(T, Y, W, 1, 128, 0);                                \
+        if (aligned && quads <= 256) JOIN_AS(T, Y, W, 1, 256, 0);                                \
+        if (aligned && quads <= 512) JOIN_AS(T, Y, W, 1, 512, 0);                                \
+        if (aligned && quads <= 1024) JOIN_AS(T, Y, W, 2, 512, 0);                               \
+        if (aligned && quads <= 2048) JOIN_AS(T, Y, W, 4, 512, 0);                               \
+        if (smem > 48 * 1024) {                                                                  \
+            cudaError_t e = cudaFuncSetAttribute(join_rmsnorm_kernel<T, Y, W, 0>,                \
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize,    \
+                                                 (int)smem);                                     \
+            if (e != cudaSuccess) return (int)e;                                                 \
+        }                                                                                        \
+        JOIN_AS(T, Y, W, 0, row_threads(width), smem);                                           \
+    } while (0)
+    if (dtype == DE_BF16) {
+        if (y_dtype == DE_BF16) {
+            if (weight_dtype == DE_BF16) JOIN(__nv_bfloat16, __nv_bfloat16, __nv_bfloat16);
+            JOIN(__nv_bfloat16, __nv_bfloat16, float);
+        }
+        if (weight_dtype == DE_BF16) JOIN(__nv_bfloat16, float, __nv_bfloat16);
+        JOIN(__nv_bfloat16, float, float);
+    }
+    if (weight_dtype == DE_BF16) JOIN(float, float, __nv_bfloat16);
+    JOIN(float, float, float);
+#undef JOIN
+#undef JOIN_AS
 }

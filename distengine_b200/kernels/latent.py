@@ -11,11 +11,13 @@ from .ops import ACTIVATIONS, _check, _i32, _need, _ptr, _stream, _tag
 
 def latent_write(q: torch.Tensor, kv: torch.Tensor, qa: torch.Tensor, freq: torch.Tensor,
                  magnitude: float, norm_weight: torch.Tensor, eps: float, heads: int, dim: int,
-                 rot: int, rank: int, pages: torch.Tensor, block_table: torch.Tensor, ctx) -> None:
+                 rot: int, rank: int, pages: torch.Tensor, block_table: torch.Tensor, ctx,
+                 adjacent: bool = False) -> None:
     """Per token: the latent c = rms_norm(kv[:, :rank]) * norm_weight and the key part kv[:, rank:]
     turned by the token's position go to the pages ([pages, 1, page, rank + rot]); every head's
     rotated query part (q rows are heads of [dim | rot]) goes, turned, to columns rank.. of its
-    head in ``qa`` (rows of heads of [rank | rot]).  ``freq`` float64 [rot / 2]; cosine and sine
+    head in ``qa`` (rows of heads of [rank | rot]).  Pairs are (i, i + rot / 2) of a rotated part, or
+    with ``adjacent`` (2i, 2i + 1).  ``freq`` float64 [rot / 2]; cosine and sine
     are multiplied by ``magnitude``."""
     n = q.shape[0]
     _need(q.stride(1) == 1 and kv.stride(1) == 1 and qa.stride(1) == 1
@@ -34,7 +36,7 @@ def latent_write(q: torch.Tensor, kv: torch.Tensor, qa: torch.Tensor, freq: torc
                                kv.data_ptr(), kv.stride(0), qa.data_ptr(), qa.stride(0),
                                ctx.positions.data_ptr(), ctx.token_slot.data_ptr(),
                                freq.data_ptr(), float(magnitude), norm_weight.data_ptr(),
-                               float(eps), heads, dim, rot, rank, pages.data_ptr(),
+                               float(eps), int(adjacent), heads, dim, rot, rank, pages.data_ptr(),
                                block_table.data_ptr(), block_table.stride(0), pages.shape[2],
                                pages.shape[0], n, ctx.status.data_ptr(), _stream()),
            "latent_write")
@@ -71,15 +73,25 @@ def experts_tiles(n: int, top: int, experts: int, segment: int = SEGMENT) -> int
     return int(library.load("experts").de_experts_tiles(n, top, experts, segment))
 
 
+SCORINGS = {"chosen_logits": 0, "corrected_scores": 1, "grouped_sigmoid": 2}
+
+
 def experts_route(h: torch.Tensor, router: torch.Tensor, bias: torch.Tensor, top: int,
                   chosen: torch.Tensor, weight: torch.Tensor,
-                  scoring: str = "chosen_logits") -> None:
+                  scoring: str = "chosen_logits", groups: int = 1, keep: int = 1,
+                  scale: float = 1.0, side: "torch.Tensor | None" = None) -> None:
     """chosen [N, top] (int32): the experts with the largest logits router h + bias (float32);
     weight [N, top] (float32): the softmax over those logits alone.  ``scoring``
     "corrected_scores": the scores are the softmax of router h over all outputs, the choice goes
-    by score + bias, and the weights are the chosen scores as they are."""
-    n, experts = h.shape[0], router.shape[0]
-    _need(scoring in ("chosen_logits", "corrected_scores"), "experts_route: unknown scoring")
+    by score + bias, and the weights are the chosen scores as they are.  "grouped_sigmoid": the
+    scores are sigmoid(router h), the choice goes by score + bias among the experts of the
+    ``keep`` best of ``groups`` equal groups (a group's value: its two largest choice scores'
+    sum), and the weights are the chosen scores over their sum (+ 1e-20) times ``scale``.
+    ``side`` float32 [N]: the router has a row more, whose logit's sigmoid goes there."""
+    n, experts = h.shape[0], router.shape[0] - (side is not None)
+    _need(scoring in SCORINGS, "experts_route: unknown scoring")
+    _need(side is None or (side.dtype == torch.float32 and side.shape == (n,)
+                           and side.is_contiguous()), "experts_route: side float32 [N]")
     _i32(chosen, "chosen")
     _need(h.stride(1) == 1 and router.dtype == bias.dtype == weight.dtype == torch.float32
           and router.is_contiguous() and router.shape[1] == h.shape[1] and bias.is_contiguous()
@@ -88,8 +100,9 @@ def experts_route(h: torch.Tensor, router: torch.Tensor, bias: torch.Tensor, top
     lib = library.load("experts")
     _check(lib.de_experts_route(_tag(h.dtype), h.data_ptr(), h.stride(0), router.data_ptr(),
                                 bias.data_ptr(), n, h.shape[1], experts, top,
-                                int(scoring == "corrected_scores"), chosen.data_ptr(),
-                                weight.data_ptr(), _stream()), "experts_route")
+                                SCORINGS[scoring], int(groups), int(keep), float(scale),
+                                chosen.data_ptr(), weight.data_ptr(), _ptr(side), _stream()),
+           "experts_route")
 
 
 def experts_group(chosen: torch.Tensor, experts: int, pair_of: torch.Tensor,
@@ -189,11 +202,19 @@ def experts_product(rows: torch.Tensor, w: torch.Tensor, pair_of: torch.Tensor,
 
 
 def experts_combine(y: torch.Tensor, weight: torch.Tensor, out: torch.Tensor,
-                    hands_on: "tuple | None" = None) -> None:
+                    hands_on: "tuple | None" = None, shared: "tuple | None" = None) -> None:
     """out[n] = sum_k weight[n, k] * y[n * top + k] in float32; out float32 [N, D].
     ``hands_on`` = (chosen [N, top], experts, h [N, D]): a pair whose choice is not below
-    ``experts`` has no row in y; it adds weight * h[n]."""
+    ``experts`` has no row in y; it adds weight * h[n].  ``shared`` = (rows [N, D], side float32
+    [N]): side[n] * rows[n] joins the sum."""
     n, top = weight.shape
+    both = (None, None)
+    if shared is not None:
+        rows, side = shared
+        _need(rows.dtype == y.dtype and rows.is_contiguous() and rows.shape == out.shape
+              and side.dtype == torch.float32 and side.shape == (n,) and side.is_contiguous(),
+              "experts_combine: shared rows [N, D] of y's dtype, side float32 [N]")
+        both = (rows.data_ptr(), side.data_ptr())
     extra = (None, 0, None, 0)
     if hands_on is not None:
         chosen, experts, h = hands_on
@@ -206,5 +227,17 @@ def experts_combine(y: torch.Tensor, weight: torch.Tensor, out: torch.Tensor,
           and weight.is_contiguous(), "experts_combine: y [N top, D], weight [N, top], out [N, D]")
     lib = library.load("experts")
     _check(lib.de_experts_combine(_tag(y.dtype), y.data_ptr(), weight.data_ptr(), n, top,
-                                  out.shape[1], out.data_ptr(), *extra, _stream()),
+                                  out.shape[1], out.data_ptr(), *extra, *both, _stream()),
            "experts_combine")
+
+
+def clipped_glu(x: torch.Tensor, out: torch.Tensor, limit: float, sharpness: float) -> None:
+    """out = g sigmoid(sharpness g) (u + 1) with g = min(x[:, :inner], limit) and u = x[:, inner:]
+    clamped to +- limit; x [N, 2 inner], out [N, inner] of one dtype."""
+    n, inner = out.shape
+    _need(x.shape == (n, 2 * inner) and x.stride(1) == 1 and out.stride(1) == 1
+          and x.dtype == out.dtype, "clipped_glu: x [N, 2 inner], out [N, inner]")
+    lib = library.load("experts")
+    _check(lib.de_clipped_glu(_tag(x.dtype), x.data_ptr(), x.stride(0), out.data_ptr(),
+                              out.stride(0), n, inner, float(limit), float(sharpness), _stream()),
+           "clipped_glu")

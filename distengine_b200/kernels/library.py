@@ -99,25 +99,37 @@ SIGNATURES: dict[str, dict[str, list]] = {
         "de_head_gate": [I, P, P, I, P, P, I, I, I, F, I, P],
         "de_mean_of_normed": [I, P, P, P, P, P, I, I, F, P],
     },
+    "ssm": {
+        "de_ssm_max_state": [], "de_ssm_chunk": [],
+        "de_ssm_prep": [I, P, I, P, I, P, P, P, P, P, L, I, P, P, P, P, P, P, I, I, I, I, I, I, P],
+        "de_ssm_walk": [I, I, P, I, P, I, P, P, P, P, P, P, P, P, L, I, P, P, P, I, I, P, I, I, I,
+                        I, I, P],
+        "de_ssm_chunk_state": [P, P, P, I, P, P, I, I, I, I, I, P],
+        "de_ssm_chunk_pass": [P, P, P, I, P, P, L, I, I, I, P],
+        "de_ssm_chunk_out": [P, P, P, I, P, P, P, I, I, I, I, I, P],
+        "de_gated_group_norm": [I, P, P, I, P, P, I, I, I, F, P, I, I, I, I, P, L, P, P, P, P, P, P],
+    },
     "latent": {
-        "de_latent_write": [I, I, P, I, P, I, P, I, P, P, P, F, P, F, I, I, I, I, P, P, I, I, I, I,
-                            P, P],
+        "de_latent_write": [I, I, P, I, P, I, P, I, P, P, P, F, P, F, I, I, I, I, I, P, P, I, I, I,
+                            I, P, P],
         "de_heads_product": [I, I, I, P, I, I, P, P, I, I, P, I, I, I, I, I, P],
     },
     "experts": {
         "de_experts_tiles": [I, I, I, I],
         "de_experts_gather": [I, P, I, P, I, I, I, P, P],
-        "de_experts_route": [I, P, I, P, P, I, I, I, I, I, P, P, P],
+        "de_experts_route": [I, P, I, P, P, I, I, I, I, I, I, I, F, P, P, P, P],
         "de_experts_group": [P, I, I, I, I, P, P, P, P],
         "de_experts_up": [I, P, I, P, P, P, I, I, I, I, P, I, P],
         "de_experts_down": [I, P, P, P, P, I, I, I, P, P],
-        "de_experts_combine": [I, P, P, I, I, I, P, P, I, P, I, P],
+        "de_experts_combine": [I, P, P, I, I, I, P, P, I, P, I, P, P, P],
+        "de_clipped_glu": [I, P, I, P, I, I, I, F, F, P],
     },
     "sublayer": {
         "de_norm_stream": [I, I, P, P, P, I, I, F, P],
         "de_gated_normed_add": [I, I, I, P, P, I, P, P, P, P, P, I, I, F, P],
         "de_depth_mix": [I, P, L, P, I, L, P, P, P],
         "de_poly_norm": [I, P, I, P, P, I, I, I, F, P],
+        "de_join_rmsnorm": [I, I, I, P, P, P, F, P, P, F, P, P, I, I, P],
     },
     "attention_decode": {
         "de_attn_decode_head_dim": [], "de_attn_decode_max_cluster": [],

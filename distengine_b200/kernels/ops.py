@@ -291,6 +291,44 @@ def gated_normed_add(y: torch.Tensor, gate: torch.Tensor, bias: torch.Tensor, we
                                    n, width, float(eps), _stream()), "gated_normed_add")
 
 
+def join_rmsnorm(resid: torch.Tensor, y: "torch.Tensor | None", branch_norm=None,
+                 vector: "torch.Tensor | None" = None, norm=None,
+                 out: "torch.Tensor | None" = None, rows: "torch.Tensor | None" = None) -> None:
+    """resid += y / sqrt(mean(y^2) + eps) * weight + vector row by row in float32, with weight and
+    eps of ``branch_norm`` (None: y as it is), y [N, width] (None: no branch) and vector float32
+    [width] (None: none); then, with ``out``, out = the RMS norm ``norm`` of the new rows.
+    ``rows`` (int32): out[i] is the norm of row rows[i], and resid stays as it is."""
+    n, width = resid.shape
+    _need(resid.dtype == torch.float32 and resid.is_contiguous() and (y is None or (
+        y.is_contiguous() and y.shape == resid.shape)), "join_rmsnorm: resid float32, y [N, width]")
+    _need(vector is None or (vector.dtype == torch.float32 and vector.is_contiguous()
+                             and vector.shape == (width,)), "join_rmsnorm: vector float32 [width]")
+    _need((norm is None) == (out is None) and (rows is None or out is not None),
+          "join_rmsnorm: a norm and its output come together")
+    if y is None:
+        branch_norm = None
+    n_out = n
+    if out is not None:
+        n_out = out.shape[0]
+        _need(out.is_contiguous() and out.shape[1] == width
+              and n_out == (n if rows is None else rows.shape[0]), "join_rmsnorm: out [.., width]")
+    if rows is not None:
+        _i32(rows, "rows")
+    weights = [w.weight for w in (branch_norm, norm) if w is not None]
+    for w in weights:
+        _need(w.shape == (width,) and _wtag(w) == _wtag(weights[0]),
+              "join_rmsnorm: both weights [width] of one dtype")
+    y_dtype = torch.float32 if y is None else y.dtype
+    dtype = out.dtype if out is not None else torch.bfloat16
+    lib = library.load("sublayer")
+    _check(lib.de_join_rmsnorm(
+        _tag(dtype), _tag(y_dtype), _wtag(weights[0]) if weights else 0, resid.data_ptr(), _ptr(y),
+        None if branch_norm is None else branch_norm.weight.data_ptr(),
+        0.0 if branch_norm is None else float(branch_norm.eps), _ptr(vector),
+        None if norm is None else norm.weight.data_ptr(), 0.0 if norm is None else float(norm.eps),
+        _ptr(out), _ptr(rows), n_out, width, _stream()), "join_rmsnorm")
+
+
 def depth_mix(history: torch.Tensor, coef: torch.Tensor, out: torch.Tensor,
               rows: "torch.Tensor | None" = None) -> None:
     """out = sum_j coef[j] * history[j]; history float32 [count, N, width] (contiguous), coef

@@ -1,4 +1,5 @@
-from . import bizetar, llama, sebilorn, vapelix, vomotar  # noqa: F401  (register the architectures)
+from . import (bizetar, llama, puripel, sebilorn, vapelix,  # noqa: F401  (register the
+               vomotar)                                     # architectures)
 from .decoder import DecoderModel, expected_tensors
 from .loading import load_model
 

@@ -53,6 +53,12 @@ class DecoderModel:
         self.final_norm = build_norm(config.final_norm(), dtype, self.device)
         first = config.embedding_norm()
         self.embedding_norm = None if first is None else build_norm(first, dtype, self.device)
+        self.plan_vectors: "torch.Tensor | None" = None
+        for index, entry in enumerate(self.plan):
+            if entry.adds_vector is not None and not (
+                    0 <= entry.adds_vector < config.plan_vectors()):
+                raise ValueError(f"plan entry {index} adds vector {entry.adds_vector}, the model "
+                                 f"has {config.plan_vectors()}")
         # the states of the stream that blocks read besides the stream itself
         self.history_depth = max((block.history_depth() for block in self.blocks), default=0)
         self.embedding: "torch.Tensor | None" = None
@@ -82,6 +88,8 @@ class DecoderModel:
                 expected[prefix + local] = tuple(shape)
                 if kind == "vector":
                     vectors.add(prefix + local)
+        if self.config.plan_vectors():
+            expected[names["plan_vectors"]] = (self.config.plan_vectors(), self.config.width)
         expected[names["output"]] = (self.config.vocabulary, self.config.width)
         # a tied output needs no tensor of its own, unless it goes by the embedding's name
         optional = ({names["output"]} - {names["embedding"]}) if self.config.tied_output else set()
@@ -91,7 +99,7 @@ class DecoderModel:
         """The kernel libraries every step of this model uses: the row-wise kernels, the product
         of its dtype for steps of few tokens, and what its parts name."""
         modules = ["core", "gemm_f32" if self.dtype == torch.float32 else "linear_small"]
-        if self.embedding_norm is not None:
+        if self.embedding_norm is not None or self.config.plan_vectors():
             modules.append("sublayer")
         for block in self.blocks:
             for part in block.parts().values():
@@ -116,6 +124,9 @@ class DecoderModel:
         if self.embedding_norm is not None:
             self.embedding_norm.load({local: tensors[names["embedding_norm"] + local]
                                       for local in self.embedding_norm.tensors()})
+        if self.config.plan_vectors():
+            self.plan_vectors = tensors[names["plan_vectors"]].to(
+                device=self.device, dtype=torch.float32).contiguous()
         if names["output"] in tensors:
             self.output = compute_matrix(tensors[names["output"]], self.dtype, self.device)
         else:
@@ -192,12 +203,19 @@ class DecoderModel:
             if entry.adds_embedding:
                 if stream.ahead is not None:
                     raise RuntimeError("a pass cannot start while a norm's work is handed ahead")
+                if stream.pending_norm is not None or stream.pending_vector is not None:
+                    stream.settle()
                 ops.residual_add(stream.resid, stream.pending, None, first)
                 stream.pending = None
+            if entry.adds_vector is not None:
+                if stream.ahead is not None:
+                    raise RuntimeError("a pass cannot start while a norm's work is handed ahead")
+                stream.add_vector(self.plan_vectors[entry.adds_vector])
             # the norm and mixer that read the stream next, for blocks that hand a norm's work to
             # the product before it
             following = None
-            if index + 1 < len(self.plan) and not self.plan[index + 1].adds_embedding:
+            if (index + 1 < len(self.plan) and not self.plan[index + 1].adds_embedding
+                    and self.plan[index + 1].adds_vector is None):
                 later = self.blocks[self.plan[index + 1].layer]
                 following = (later.mixer_norm, later.mixer)
             self.blocks[entry.layer].forward(stream, ctx, caches[index], following=following)

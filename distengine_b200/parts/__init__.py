@@ -1,4 +1,4 @@
-from . import (attention, block, chunk_attention, experts, latent_attention,  # noqa: F401
+from . import (attention, block, chunk_attention, experts, latent_attention, mamba2,  # noqa: F401
                mlp, norm, parallel, recurrent, rope, sink_attention, token_side,
                window_attention)  # (register the built-in kinds)
 from .base import (Block, FeedForward, Mixer, Norm, PagedKVSpec, Part, PositionEncoding,

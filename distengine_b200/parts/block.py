@@ -4,6 +4,8 @@ by the next norm.  A layer without a feed-forward is the first half only.
 
 ``parallel_norms``: both branches read the same x (see ``ParallelNormsBlock``).
 
+``sandwich``: a norm before and one after each sublayer (see ``SandwichBlock``).
+
 ``sublayer_norm``: the norm stands on a sublayer's output, the sublayers read x itself, with an
 optional gate on every sublayer's result and an optional average over the depth (see
 ``SublayerNormBlock``)."""
@@ -13,7 +15,7 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from .base import Block, Part, register_block
+from .base import Block, Part, build_norm, register_block
 from .context import CacheBinding, ResidualStream, StepContext
 
 
@@ -96,6 +98,49 @@ class ParallelNormsBlock(Block):
 
 
 register_block("parallel_norms", ParallelNormsBlock)
+
+
+class SandwichBlock(Block):
+    """x <- x + after1(mixer(norm1(x))); x <- x + after2(feed_forward(norm2(x))): an RMS norm before
+    and one after each sublayer.  The norm after a sublayer, the sum and the norm that reads the
+    stream next are one kernel (``ops.join_rmsnorm``): the block leaves the branch pending together
+    with its norm.  ``mixer_after`` and ``feed_forward_after``: the specs of the norms after the
+    sublayers (kind ``branch_rmsnorm``; roles of the same names).  A layer without a feed-forward
+    is the first half only."""
+
+    def __init__(self, mixer, feed_forward, mixer_norm, feed_forward_norm, side_input=None, *,
+                 mixer_after, feed_forward_after=None) -> None:
+        super().__init__(mixer, feed_forward, mixer_norm, feed_forward_norm, side_input)
+        if side_input is not None or (feed_forward is None) != (feed_forward_after is None):
+            raise ValueError("sandwich: no side input, and a norm after the feed-forward if there "
+                             "is one")
+        self.mixer_after = build_norm(mixer_after, mixer.dtype, mixer.device)
+        self.feed_forward_after = None
+        if feed_forward_after is not None:
+            self.feed_forward_after = build_norm(feed_forward_after, mixer.dtype, mixer.device)
+
+    def parts(self):
+        parts = super().parts()
+        for role in ("mixer_after", "feed_forward_after"):
+            if getattr(self, role) is not None:
+                parts[role] = getattr(self, role)
+        return parts
+
+    def forward(self, stream: ResidualStream, ctx: StepContext, cache: "CacheBinding | None",
+                following=None) -> None:
+        if stream.ahead is not None:
+            raise RuntimeError("a sandwich block runs its norms itself")
+        h = self.mixer_norm.forward(stream, ctx)
+        stream.pending = self.mixer.forward(h, ctx, cache)
+        stream.pending_norm = self.mixer_after
+        if self.feed_forward is None:
+            return
+        h = self.feed_forward_norm.forward(stream, ctx)
+        stream.pending = self.feed_forward.forward(h, ctx)
+        stream.pending_norm = self.feed_forward_after
+
+
+register_block("sandwich", SandwichBlock)
 
 
 class ResidualGate(Part):

@@ -159,11 +159,17 @@ class ResidualStream:
     A norm folds ``pending`` into ``resid`` in the same kernel that normalises, so the sum is
     formed in 32-bit and costs no pass over memory of its own.  ``ahead``: the last product
     already added its result and did the next norm's work (``NormAhead``); that norm hands out
-    its result instead of running."""
+    its result instead of running.
+
+    ``pending_norm``: a norm (``weight``, ``eps``) that the pending branch output passes on its way
+    into the stream.  ``pending_vector``: a vector that every row of the stream is still to
+    receive after that.  A norm that cannot fold these calls ``settle`` first."""
 
     def __init__(self, resid: torch.Tensor) -> None:
         self.resid = resid                      # float32 [N, width]
         self.pending: "torch.Tensor | None" = None
+        self.pending_norm: "Any | None" = None
+        self.pending_vector: "torch.Tensor | None" = None
         self.ahead: "NormAhead | None" = None
         # the stream's rounding to the activation dtype, where the kernel that last wrote the
         # stream left one (blocks whose sublayers read the stream itself)
@@ -172,3 +178,16 @@ class ResidualStream:
         # blocks that mix the stream over the depth; ``history_count`` of them are filled
         self.history: "torch.Tensor | None" = None
         self.history_count = 0
+
+    def add_vector(self, vector: torch.Tensor) -> None:
+        if self.pending_vector is not None:
+            self.settle()
+        self.pending_vector = vector
+
+    def settle(self) -> None:
+        """Bring everything pending into the stream now."""
+        if self.pending is None and self.pending_vector is None:
+            return
+        from ..kernels import ops
+        ops.join_rmsnorm(self.resid, self.pending, self.pending_norm, self.pending_vector)
+        self.pending = self.pending_norm = self.pending_vector = None

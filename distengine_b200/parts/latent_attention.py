@@ -5,8 +5,9 @@ share).
     cq = rms_norm(W_dq x) * n_q ;  q = W_uq cq            per head [key_dim plain | rotary_dim turned]
     [c' | kr] = W_dkv x ;  c = rms_norm(c') * n_kv         c [kv_rank], kr [rotary_dim]
     k_h = W_uk[h] c ;  v_h = W_uv[h] c
-    score_h(i, j) = (q_h,plain(i) . k_h(j) + turn(q_h,rot(i)) . turn(kr(j))) * scale ;  j <= i
-    out = W_o [ heads' weighted sums of v_h * sigmoid(W_g x) ]
+    score_h(i, j) = (q_h,plain(i) . k_h(j) + turn(q_h,rot(i)) . turn(kr(j))) * scale
+        for j <= i, with ``window`` (not None) also i - j < window
+    out = W_o [ heads' weighted sums of v_h * sigmoid(W_g x) ]      (without ``gated``: no W_g)
 
 Run in the folded form, which reads nothing but [c | turn(kr)] of a key:
 q'_h = W_uk[h]^T q_h,plain, score = (q'_h . c + turn(q_h,rot) . turn(kr)) * scale, the weighted sum
@@ -14,7 +15,7 @@ is taken over c and W_uv[h] is applied to it afterwards.  That is attention with
 of size kv_rank + rotary_dim whose values are the first kv_rank features of its keys, which the
 kernels of ``csrc/attention_chunk.cu`` run; the per-head products are ``kernels.latent``.
 
-Turning: the pair (i, i + rotary_dim / 2) of the rotated part by the angle position * f_i, with
+Turning: the pair (i, i + rotary_dim / 2) of the rotated part (with ``adjacent`` (2i, 2i + 1)) by the angle position * f_i, with
 f_i = theta^(-2i / rotary_dim).  ``scaling`` = (factor, original, fast, slow) stretches the slow
 frequencies: with d(t) = rotary_dim * ln(original / (2 pi t)) / (2 ln theta),
 lo = max(floor(d(fast)), 0), hi = min(ceil(d(slow)), rotary_dim - 1) and the ramp
@@ -74,8 +75,12 @@ class LatentAttention(Mixer):
 
     def __init__(self, width: int, heads: int, key_dim: int, rotary_dim: int, value_dim: int,
                  q_rank: int, kv_rank: int, scale: float, theta: float, eps: float,
-                 dtype: torch.dtype, device: torch.device, scaling=None) -> None:
+                 dtype: torch.dtype, device: torch.device, scaling=None,
+                 window: "int | None" = None, adjacent: bool = False, gated: bool = True) -> None:
         super().__init__(dtype, device)
+        if window is not None and window <= 0:
+            raise ValueError(f"latent_attention: window must be positive or None, got {window}")
+        self.window, self.adjacent, self.gated = window, adjacent, gated
         if rotary_dim % 2 or rotary_dim < 0:
             raise ValueError(f"latent_attention: rotary_dim ({rotary_dim}) must be even")
         if kv_rank > MAX_RANK or kv_rank + rotary_dim > MAX_ROW:
@@ -87,24 +92,29 @@ class LatentAttention(Mixer):
         freq, self.magnitude = stretched_frequencies(theta, rotary_dim, scaling)
         self.freq = freq.to(device)
         self.row = kv_rank + rotary_dim              # what a key's row in the pages holds
-        self.key = f"latent_attention/{heads}/{kv_rank}/{rotary_dim}"
+        self.key = f"latent_attention/{heads}/{kv_rank}/{rotary_dim}/{window or 0}"
         # prompt portions on the tensor cores: one key/value head of `row` features
         self.launcher = None
         if uses_tensor_cores(dtype, self.row) and self.row <= MAX_HEAD_DIM:
-            self.launcher = AttentionLauncher(dtype, heads, 1, self.row, self.scale, None, device)
+            self.launcher = AttentionLauncher(dtype, heads, 1, self.row, self.scale, window,
+                                              device)
 
     def tensors(self):
         d, h = self.width, self.heads
-        return {"dq": ((self.q_rank, d), "matrix"), "dq.norm": ((self.q_rank,), "vector"),
-                "uq": ((h * (self.dim + self.rot), self.q_rank), "matrix"),
-                "dkv": ((self.row, d), "matrix"), "dkv.norm": ((self.rank,), "vector"),
-                "uk": ((h * self.dim, self.rank), "matrix"),
-                "uv": ((h * self.dv, self.rank), "matrix"),
-                "g": ((h * self.dv, d), "matrix"), "o": ((d, h * self.dv), "matrix")}
+        out = {"dq": ((self.q_rank, d), "matrix"), "dq.norm": ((self.q_rank,), "vector"),
+               "uq": ((h * (self.dim + self.rot), self.q_rank), "matrix"),
+               "dkv": ((self.row, d), "matrix"), "dkv.norm": ((self.rank,), "vector"),
+               "uk": ((h * self.dim, self.rank), "matrix"),
+               "uv": ((h * self.dv, self.rank), "matrix"),
+               "o": ((d, h * self.dv), "matrix")}
+        if self.gated:
+            out["g"] = ((h * self.dv, d), "matrix")
+        return out
 
     def load(self, tensors):
-        stacked, offsets = stack_segments([tensors["dq"], tensors["dkv"], tensors["g"]])
-        self.kv_col, self.g_col = offsets[1], offsets[2]
+        mats = [tensors["dq"], tensors["dkv"]] + ([tensors["g"]] if self.gated else [])
+        stacked, offsets = stack_segments(mats)
+        self.kv_col, self.g_col = offsets[1], offsets[2] if self.gated else 0
         self.w_in = compute_matrix(stacked, self.dtype, self.device)
         self.w_uq = compute_matrix(tensors["uq"], self.dtype, self.device)
         h = self.heads
@@ -126,7 +136,7 @@ class LatentAttention(Mixer):
         return mine + (self.launcher.module, ("attention_simt", ())) + wide
 
     def cache_spec(self):
-        return PagedKVSpec(1, self.row, value_dim=self.rank, values_in_keys=True)
+        return PagedKVSpec(1, self.row, self.window, value_dim=self.rank, values_in_keys=True)
 
     @property
     def prepare_key(self) -> str:
@@ -172,7 +182,7 @@ class LatentAttention(Mixer):
         folded = ctx.buffer("latent_attention.folded", (n, H * self.row))
         lk.latent_write(q, proj[:, self.kv_col: self.kv_col + self.row], folded, self.freq,
                         self.magnitude, self.n_kv, self.eps, H, self.dim, self.rot, self.rank,
-                        cache.k_pages, cache.block_table, ctx)
+                        cache.k_pages, cache.block_table, ctx, adjacent=self.adjacent)
         lk.heads_product(q, self.dim + self.rot, self.w_uk_t, folded, self.row)
         if ctx.notes[self.key] == -1:
             sums = ctx.buffer("latent_attention.sums", (n, H * self.row))
@@ -182,12 +192,13 @@ class LatentAttention(Mixer):
         if ctx.notes[self.key] == 0:
             rk.chunk_attention_decode(folded, mixed, cache.k_pages, cache.k_pages,
                                       cache.block_table, None, None, H, 1, self.row, self.rank,
-                                      self.scale, 0, ctx, v_stride=self.row)
+                                      self.scale, 0, ctx, window=self.window or 0,
+                                      v_stride=self.row)
         else:
             rk.chunk_attention(folded, mixed, cache.k_pages, cache.k_pages, cache.block_table,
                                ctx.arrays[self.key + "/items"], None, None, H, 1, self.row,
                                self.rank, self.scale, 0, ctx, tile_rows=ctx.notes[self.key],
-                               v_stride=self.row)
+                               window=self.window or 0, v_stride=self.row)
         return self._finish(mixed, self.rank, proj, ctx)
 
     def _finish(self, sums: torch.Tensor, stride: int, proj: torch.Tensor,
@@ -196,8 +207,8 @@ class LatentAttention(Mixer):
         W_uv[h], the gate and W_o."""
         n, H = sums.shape[0], self.heads
         context = ctx.buffer("latent_attention.context", (n, H * self.dv))
-        lk.heads_product(sums, stride, self.w_uv, context, self.dv,
-                         gate=proj[:, self.g_col: self.g_col + H * self.dv])
+        gate = proj[:, self.g_col: self.g_col + H * self.dv] if self.gated else None
+        lk.heads_product(sums, stride, self.w_uv, context, self.dv, gate=gate)
         out = ctx.buffer("latent_attention.out", (n, self.width))
         ops.linear(context, self.w_o, out=out, status=ctx.status)
         return out

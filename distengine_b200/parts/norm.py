@@ -8,6 +8,9 @@ the activation dtype, then times the weight.  The block's residual sums
 its own root mean square; the weight still spans the row.  ``tensor``: the local name of the
 weight (architectures differ in it).
 
+``branch_rmsnorm``: the norm on a branch's output before it joins the stream.  It has no kernel of
+its own: the norm that reads the stream next does its work (``ResidualStream.pending_norm``).
+
 ``layernorm``: (x - mean) / sqrt(mean of squared deviations + eps) * weight + bias, the statistics
 in float32 over the whole row; ``tensor`` and ``bias`` are the local names of its two vectors.  The
 mean does not commute with a matrix product, so this norm never rides on the products around it.
@@ -53,6 +56,14 @@ class RMSNorm(Norm):
                                "result is stream.ahead.result()")
         n_out = stream.resid.shape[0] if rows is None else rows.shape[0]
         out = ctx.buffer(out_name, (n_out, self.width))
+        if stream.pending_norm is not None or stream.pending_vector is not None:
+            if self.groups == 1:         # the branch's norm, the sums and this norm in one kernel
+                ops.join_rmsnorm(stream.resid, stream.pending, stream.pending_norm,
+                                 stream.pending_vector, self, out, rows)
+                if rows is None:
+                    stream.pending = stream.pending_norm = stream.pending_vector = None
+                return out
+            stream.settle()
         ops.add_rmsnorm(stream.resid, stream.pending, self.weight, self.eps, out, rows,
                         groups=self.groups)
         if rows is None:
@@ -71,6 +82,18 @@ class RMSNorm(Norm):
             rows = ctx.buffer("norm.stream_rows", tuple(stream.resid.shape))
         ops.norm_stream(stream.resid, self.weight, self.eps, rows)
         stream.rows = rows
+
+
+class BranchNorm(RMSNorm):
+    def __init__(self, width: int, eps: float, dtype: torch.dtype, device: torch.device,
+                 tensor: str = "weight") -> None:
+        super().__init__(width, eps, dtype, device, tensor=tensor)
+
+    def kernel_modules(self):
+        return ("sublayer",)
+
+    def forward(self, stream, ctx, rows=None, out_name="norm.out"):
+        raise RuntimeError("a branch's norm stands on the branch's output, not on the stream")
 
 
 class LayerNorm(Norm):
@@ -94,6 +117,8 @@ class LayerNorm(Norm):
                 out_name: str = "norm.out") -> torch.Tensor:
         if stream.ahead is not None:
             raise RuntimeError("a layer norm's work cannot be handed to the product before it")
+        if stream.pending_norm is not None or stream.pending_vector is not None:
+            stream.settle()
         n_out = stream.resid.shape[0] if rows is None else rows.shape[0]
         out = ctx.buffer(out_name, (n_out, self.width))
         ops.add_layernorm(stream.resid, stream.pending, self.weight, self.bias, self.eps, out, rows)
@@ -103,4 +128,5 @@ class LayerNorm(Norm):
 
 
 register_norm("rmsnorm", RMSNorm)
+register_norm("branch_rmsnorm", BranchNorm)
 register_norm("layernorm", LayerNorm)
