@@ -1,7 +1,8 @@
 """Decode and prefill throughput of the engine on one B200, random weights.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
-                    [--workload headline|mixed|long|fp32|vomotar|sebilorn|vapelix|bizetar] [--layers L]
+                    [--workload headline|mixed|long|fp32|vomotar|sebilorn|vapelix|bizetar
+                     |puripel] [--layers L]
 
 The default (``headline``) has the TinyLlama-1.1B layer sizes in bfloat16.  A step is one decode
 step of a batch of 8 requests whose prompts of 512 tokens are in the cache; K steps are timed with
@@ -52,6 +53,10 @@ Other workloads, each with its own line (the number of layers is named beside th
   same width and vocabulary, beside Sebilorn and Llama with the same number of layers: decode at
   batch 8 and 64 and a prompt of 2,048 tokens, and every kernel of the design alone against its
   roofline, each beside the like kernel of the other models.
+* ``puripel``: the Puripel architecture (Mamba-2 in three layers of four, windowed latent attention
+  in the others, a norm before and after every sublayer, experts chosen by groups beside a shared
+  one) at the same width and vocabulary, beside Vapelix, Sebilorn and Llama with the same number
+  of layers, in the same way.
 """
 
 from __future__ import annotations
@@ -1460,6 +1465,377 @@ def workload_bizetar(args, warmup: int, steps: int) -> int:
     return 0
 
 
+def puripel_shape(layers: int) -> dict:
+    """A Puripel model of the headline's width and vocabulary: Mamba-2 (64 heads of 64 values on
+    states of 128 rows, 8 groups: an inner width of twice the model's) in three layers of four,
+    latent attention of ``vapelix_shape``'s sizes with a window of 1,024 in every fourth; 16
+    experts of 1,024 inner features in 4 groups, 4 a token, beside a shared one of 1,024 in every
+    layer.  No loop, so that the layer runs equal the other models'."""
+    latent = {"heads": 16, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": 768, "kv_rank": 192,
+              "scale": 192 ** -0.5, "rot": {"dims": 64, "base": 500000.0}, "mask": {"size": 1024}}
+    mamba = {"heads": 64, "groups": 8, "state": 128, "vdim": 64, "conv": 4, "norm_groups": 8}
+    mlp = {"kind": "moe", "expert": {"ff": 1024, "limit": 7.0},
+           "shared": {"ff": 1024, "limit": 7.0},
+           "router": {"experts": 16, "top": 4, "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+    return {"architecture": "Puripel", "vocab": MODEL["vocab_size"], "width": MODEL["hidden_size"],
+            "norm": {"eps": 1e-6},
+            "layers": [{"type": "latent_attention", "mixer": latent, "mlp": mlp} if i % 4 == 0 else
+                       {"type": "mamba2", "mixer": mamba, "mlp": mlp} for i in range(layers)]}
+
+
+def puripel_folder(layers: int) -> str:
+    from distengine_b200.weights import write_random_model
+    folder = os.path.join(tempfile.gettempdir(), f"distengine_b200-bench-{os.getuid()}",
+                          f"puripel-shape-{layers}-layers-seed0-bf16")
+    marker = os.path.join(folder, ".complete")
+    if not os.path.isfile(marker):
+        print("[bench] writing the random-weights model folder ...", file=sys.stderr, flush=True)
+        write_random_model(puripel_shape(layers), folder, seed=0, dtype="bfloat16",
+                           norm_init="uniform")
+        with open(marker, "w") as handle:
+            handle.write("ok")
+    return folder
+
+
+class KernelBench:
+    """Times kernels alone (CUDA events, L2 flushed before every timed run, the median of ten) and
+    notes each beside its roofline and the like kernel of the other models."""
+
+    def __init__(self, peak: dict, device: str = "cuda:0") -> None:
+        import torch
+        self.torch, self.peak, self.device = torch, peak, device
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device=device)
+        self.fp32_peak = 148 * 128 * 2 * 1.965e9      # fused multiply-adds of the CUDA cores
+        self.rows: list[dict] = []
+
+    def context(self, lens, pos0):
+        """What the kernels read of a step of sequences of ``lens`` tokens at ``pos0``."""
+        from types import SimpleNamespace
+        import numpy as np
+        torch, dev = self.torch, self.device
+        lens, pos0 = (np.asarray(a, dtype=np.int32) for a in (lens, pos0))
+        qstart = (np.cumsum(lens) - lens).astype(np.int32)
+        seq = np.repeat(np.arange(len(lens), dtype=np.int32), lens)
+        slots = np.arange(len(lens), dtype=np.int32)
+        pos = pos0[seq] + np.arange(lens.sum(), dtype=np.int32) - qstart[seq]
+        d = lambda a: torch.from_numpy(np.ascontiguousarray(a, dtype=np.int32)).to(dev)
+        return SimpleNamespace(n_seqs=len(lens), token_seq=d(seq), token_slot=d(slots[seq]),
+                               positions=d(pos), seq_slot=d(slots), seq_qstart=d(qstart),
+                               seq_qlen=d(lens), seq_pos0=d(pos0),
+                               host=SimpleNamespace(seq_qlen=lens, seq_pos0=pos0,
+                                                    seq_qstart=qstart, seq_slot=slots),
+                               status=torch.zeros(1, dtype=torch.int32, device=dev))
+
+    def prepare(self, ctx, part) -> None:
+        """The step arrays and notes that ``part`` (anything with ``prepare``) adds."""
+        import numpy as np
+        from distengine_b200.parts.context import StepPrep, Workspace
+        torch, dev = self.torch, self.device
+        prep = StepPrep(ctx.host)
+        part(prep)
+        workspace = Workspace(torch.device(dev))
+        ctx.notes = prep.notes
+        ctx.arrays = {k: torch.from_numpy(np.ascontiguousarray(v, dtype=np.int32)).to(dev)
+                      for k, v in prep.extra.items()}
+        ctx.buffer = lambda name, shape, dt=None, zero=False: workspace.get(
+            name, shape, dt or torch.bfloat16, zero)
+
+    def time(self, fn, repeats: int = 10) -> float:
+        torch = self.torch
+        for _ in range(3):
+            fn()
+        times = []
+        for _ in range(repeats):
+            self.flush.zero_()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            times.append(a.elapsed_time(b) * 1e3)
+        return statistics.median(times)
+
+    def record(self, name, case, fn, bytes_=0, flops=0, tensor_flops=0, like="") -> None:
+        us = self.time(fn)
+        bounds = {"hbm": bytes_ / (self.peak["hbm_gbs"] * 1e3),
+                  "fp32 fma": flops / self.fp32_peak * 1e6,
+                  "tensor": tensor_flops / (self.peak["bf16_tflops"] * 1e12) * 1e6}
+        bound = max(bounds, key=bounds.get)
+        self.rows.append({"kernel": name, "case": case, "us": round(us, 1), "like": like,
+                          "bound": bound, "roofline_us": round(bounds[bound], 1),
+                          "frac": round(bounds[bound] / us, 3)})
+
+
+def puripel_kernels(peak: dict) -> list[dict]:
+    """The design's kernels alone at the sizes of ``puripel_shape``, for a prompt of 2,048 tokens
+    and for a decode step of 64 sequences at position 1,500, each beside the like kernel of the
+    other models in the same run (``like``): windowed attention over the latent beside the same
+    without a window and the turn of neighbours beside that of halves (Vapelix's), the state-space
+    mixer beside the state scan and its preparation at a state of the same size (Vomotar's and
+    Sebilorn's), the experts' kernels beside Bizetar's forms, the norms around a sublayer beside
+    the RMS norm."""
+    import torch
+    from types import SimpleNamespace
+    from distengine_b200.kernels import latent as lk
+    from distengine_b200.kernels import ops, ssm
+    from distengine_b200.kernels import recurrent as rk
+    from distengine_b200.kernels.attention import AttentionLauncher
+    from distengine_b200.parts.latent_attention import stretched_frequencies
+    from distengine_b200.parts.mamba2 import Mamba2
+    dev, bf16 = "cuda:0", torch.bfloat16
+    kb = KernelBench(peak, dev)
+    shape = puripel_shape(2)
+    m, mm, mlp = (shape["layers"][0]["mixer"], shape["layers"][1]["mixer"],
+                  shape["layers"][1]["mlp"])
+    width, page = MODEL["hidden_size"], PAGE
+    H, dim, rot, dv, rank = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    row, window = rank + rot, m["mask"]["size"]
+    freq = stretched_frequencies(m["rot"]["base"], rot)[0].to(dev)
+    w = lambda *s: (torch.randn(*s, device=dev) / s[-1] ** 0.5).to(bf16)
+    f = lambda *s: torch.randn(*s, device=dev)
+    for case, lens, pos0 in (("prompt of 2,048", [2048], [0]),
+                             ("decode, 64 sequences", [1] * 64, [1500] * 64)):
+        ctx = kb.context(lens, pos0)
+        n, s = int(sum(lens)), len(lens)
+        longest = max(p + l for p, l in zip(pos0, lens))
+        pages_seq = (longest + page - 1) // page
+        table = torch.arange(s * pages_seq, dtype=torch.int32, device=dev).view(s, pages_seq)
+        # ---- latent attention with a window
+        q, kv = f(n, H * (dim + rot)).to(bf16), f(n, row).to(bf16)
+        folded = torch.empty(n, H * row, dtype=bf16, device=dev)
+        pages = f(s * pages_seq, 1, page, row).to(bf16)
+        n_kv = torch.rand(rank, device=dev).to(bf16)
+        for name, adjacent, like in (("latent_write (neighbours turned)", True, "latent_write"),
+                                     ("latent_write (other models)", False, "")):
+            kb.record(name, case, lambda: lk.latent_write(
+                q, kv, folded, freq, 1.0, n_kv, 1e-6, H, dim, rot, rank, pages, table, ctx,
+                adjacent=adjacent), bytes_=n * (H * rot * 4 + 2 * row * 2), like=like)
+        mixed = torch.empty(n, H * rank, device=dev)
+        sums16 = torch.empty(n, H * row, dtype=bf16, device=dev)
+        for name, size, like in ((f"attention over the latent, window {window}", window,
+                                  "attention over the latent"),
+                                 ("attention over the latent (other models)", None, "")):
+            reach = size or 1 << 30
+            keys = sum(min(p + i + 1, reach) for p, l in zip(pos0, lens) for i in range(l))
+            read = sum(min(p + l, reach + l - 1) for p, l in zip(pos0, lens))
+            if n == s:
+                kb.record(name, case, lambda: rk.chunk_attention_decode(
+                    folded, mixed, pages, pages, table, None, None, H, 1, row, rank, m["scale"],
+                    0, ctx, window=size or 0, v_stride=row),
+                    bytes_=read * row * 2 + n * H * (row * 2 + rank * 4),
+                    flops=2 * keys * H * (row + rank), like=like)
+            else:
+                launcher = AttentionLauncher(bf16, H, 1, row, m["scale"], size)
+                kb.prepare(ctx, lambda prep: launcher.prepare(prep, allow_decode=False))
+                kb.record(name, case, lambda: launcher.run(folded, sums16, pages, pages, table,
+                                                           ctx),
+                          bytes_=read * row * 2 + n * H * row * 4,
+                          tensor_flops=2 * keys * H * 2 * row, like=like)
+        sums, a_head = (mixed, rank) if n == s else (sums16, row)
+        w_uv, context = w(H, dv, rank), torch.empty(n, H * dv, dtype=bf16, device=dev)
+        gate = f(n, H * dv).to(bf16)
+        for name, g, like in (("heads_product (values)", None, "heads_product"),
+                              ("heads_product (other models: gated)", gate, "")):
+            kb.record(name, case, lambda: lk.heads_product(sums, a_head, w_uv, context, dv,
+                                                           gate=g),
+                      bytes_=n * H * (rank * (4 if n == s else 2) + dv * (4 if g is not None
+                                                                          else 2))
+                      + H * rank * dv * 2, flops=2 * n * H * dv * rank, like=like)
+        # ---- Mamba-2 beside the state scan with a state of the same size
+        sz = ssm.Sizes(mm["heads"], mm["groups"], mm["state"], mm["vdim"], mm["conv"])
+        C, S = sz.channels, sz.state_size
+        wt = ssm.Weights(f(sz.taps, C), f(C), f(sz.heads) - 2, f(sz.heads), f(sz.heads))
+        proj = f(n, sz.inner + C + sz.heads).to(bf16)
+        z, xbc, dt = proj.split([sz.inner, C, sz.heads], dim=1)
+        state = torch.zeros(s, sz.slot_size, device=dev)
+        y, norm_w = torch.empty(n, sz.inner, device=dev), torch.rand(sz.inner, device=dev)
+        gated = torch.empty(n, sz.inner, dtype=bf16, device=dev)
+        moved = n * (C * 2 + sz.inner * 4) + 2 * s * S * 4
+        if n == s:
+            kb.record("ssm step (convolution, state, read-out)", case,
+                      lambda: ssm.step(sz, wt, xbc, dt, state, y, ctx),
+                      bytes_=moved + n * (sz.taps - 1) * C * 4, flops=5 * n * S,
+                      like="state_scan")
+        else:
+            mixer = Mamba2(width, sz.heads, sz.groups, sz.state_dim, sz.value_dim, sz.taps,
+                           mm["norm_groups"], 1e-6, bf16, torch.device(dev))
+            kb.prepare(ctx, mixer.prepare)
+            ready, rates = torch.empty(n, C, device=dev), torch.empty(n, 2 * sz.heads, device=dev)
+            items, portions = ctx.arrays["mamba2/items"], ctx.arrays["mamba2/portions"]
+            k = items.shape[0]
+            states, decays = torch.empty(k, S, device=dev), torch.empty(k, sz.heads, device=dev)
+            kb.record("ssm prep (convolution with bias, rates)", case,
+                      lambda: ssm.prep(sz, wt, xbc, dt, state, ready, rates, ctx),
+                      bytes_=n * C * (2 + 4), like="delta_prep")
+
+            def chunks():
+                ssm.chunk_state(sz, ready, rates, items, states, decays)
+                ssm.chunk_pass(sz, states, decays, portions, state, ctx)
+                ssm.chunk_out(sz, wt, ready, rates, items, states, y)
+            # multiply-adds: the state's update and read-out, c . b and the sum over the chunk
+            fma = n * (2 * S + sz.groups * ssm.CHUNK * sz.state_dim
+                       + sz.heads * ssm.CHUNK * sz.value_dim // 2)
+            kb.record("ssm chunks (three kernels)", case, chunks,
+                      bytes_=n * (C + sz.inner) * 4 + 2 * s * S * 4, flops=2 * fma,
+                      like="state_scan")
+            kb.record("ssm chunk_state", case,
+                      lambda: ssm.chunk_state(sz, ready, rates, items, states, decays),
+                      bytes_=n * C * 4 + k * S * 4, flops=2 * n * S)
+            kb.record("ssm chunk_pass", case,
+                      lambda: ssm.chunk_pass(sz, states, decays, portions, state, ctx),
+                      bytes_=2 * k * S * 4)
+            kb.record("ssm chunk_out", case,
+                      lambda: ssm.chunk_out(sz, wt, ready, rates, items, states, y),
+                      bytes_=n * (C + sz.inner) * 4 + k * S * 4, flops=2 * (fma - n * S))
+        kb.record("gated_group_norm (kept rows moved on)", case,
+                  lambda: ssm.gated_group_norm(y, z, norm_w, mm["norm_groups"], 1e-6, gated, ctx,
+                                               keep=(sz, xbc, state)),
+                  bytes_=n * sz.inner * 8 + s * (sz.taps - 1) * C * 8, like="head_gate")
+        sh, dk, sv = sz.heads, sz.state_dim, sz.value_dim
+        qn, kn, vv = f(n, sh * dk), f(n, sh * dk), f(n, sh * sv)
+        decay, o = torch.rand(sh, device=dev), torch.empty(n, sh * sv, device=dev)
+        kb.record("state_scan (other models: retention, a state of this size)", case,
+                  lambda: rk.state_scan(qn, kn, vv, state, o, sh, sh, dk, sv, ctx, decay=decay),
+                  bytes_=2 * s * S * 4 + n * sh * (2 * dk + 2 * sv) * 4, flops=n * S * 5)
+        dh, dd = 16, 128                       # the delta rule's preparation at 6,144 channels
+        dC = 3 * dh * dd
+        dproj, da = f(n, dC + dh).to(bf16), f(n, dh * dd)
+        dstate = torch.zeros(s, dh * dd * dd + 3 * dC, device=dev)
+        outs = [torch.empty(n, dh * dd, device=dev) for _ in range(3)]
+        dbeta, dg = torch.empty(n, dh, device=dev), torch.empty(n, dh * dd, device=dev)
+        taps, dvec, dlog = f(dC, 4), f(dh * dd), f(dh)
+        kb.record("delta_prep (other models: convolution, unit norms, decays)", case,
+                  lambda: rk.delta_prep(dproj, da, taps, dvec, dlog, dstate, dh * dd * dd, ctx,
+                                        *outs, dbeta, dg, dh, dh, dd, dd, dC),
+                  bytes_=n * (dC * 2 + dh * dd * 5 * 4))
+        og, gg = f(n, sz.inner), f(n, sz.inner)
+        vec = torch.rand(sv, device=dev)
+        kb.record("head_gate (other models)", case,
+                  lambda: rk.head_gate(og, gg, vec, gated, sh, sv, 1e-6),
+                  bytes_=n * sz.inner * (4 + 4 + 2))
+        # ---- norms around a sublayer
+        resid, branch = f(n, width), f(n, width).to(bf16)
+        norm = SimpleNamespace(weight=torch.rand(width, device=dev).to(bf16), eps=1e-6)
+        normed = torch.empty(n, width, dtype=bf16, device=dev)
+        kb.record("join_rmsnorm (branch norm, sum, next norm)", case,
+                  lambda: ops.join_rmsnorm(resid, branch, norm, None, norm, normed),
+                  bytes_=n * width * (4 + 4 + 2 + 2), like="add_rmsnorm")
+        kb.record("add_rmsnorm (other models)", case,
+                  lambda: ops.add_rmsnorm(resid, branch, norm.weight, 1e-6, normed),
+                  bytes_=n * width * (4 + 4 + 2 + 2))
+        # ---- experts
+        r, eff, sff = mlp["router"], mlp["expert"]["ff"], mlp["shared"]["ff"]
+        E, top, groups = r["experts"], r["top"], r["groups"]
+        x = f(n, width).to(bf16)
+        router, corr = f(E + 1, width) / width ** 0.5, 0.01 * f(E)
+        up, down = w(E, 2 * eff, width), w(E, width, eff)
+        seg = lk.SEGMENT_TENSOR
+        tiles = lk.experts_tiles(n, top, E, seg)
+        chosen = torch.empty(n, top, dtype=torch.int32, device=dev)
+        weight, side = torch.empty(n, top, device=dev), torch.empty(n, device=dev)
+        pair_of = torch.empty(tiles * seg, dtype=torch.int32, device=dev)
+        tile_expert = torch.empty(tiles, dtype=torch.int32, device=dev)
+        slot_of = torch.empty(n * top, dtype=torch.int32, device=dev)
+        route_bytes = n * width * 2 + (E + 1) * width * 4
+        kb.record("experts_route (scores over all outputs; other models)", case,
+                  lambda: lk.experts_route(x, router[:E], corr, top, chosen, weight,
+                                           "corrected_scores"),
+                  bytes_=route_bytes, flops=2 * n * E * width)
+        kb.record("experts_route (groups, shared expert's factor)", case,
+                  lambda: lk.experts_route(x, router, corr, top, chosen, weight,
+                                           "grouped_sigmoid", groups["count"], groups["keep"],
+                                           r["scale"], side),
+                  bytes_=route_bytes, flops=2 * n * (E + 1) * width, like="experts_route")
+        kb.record("experts_group", case,
+                  lambda: lk.experts_group(chosen, E, pair_of, tile_expert, slot_of, seg),
+                  bytes_=n * top * 12 + tiles * seg * 4, like="experts_group")
+        rows = torch.empty(tiles * seg, width, dtype=bf16, device=dev)
+        both = torch.zeros(tiles * seg, 2 * eff, dtype=bf16, device=dev)
+        inner = torch.empty(tiles * seg, eff, dtype=bf16, device=dev)
+        ye, eo = torch.empty(n * top, width, dtype=bf16, device=dev), torch.empty(n, width,
+                                                                                device=dev)
+        weights_read = min(E, n * top) * eff * width * 2
+        pairs = n * top
+        kb.record("experts_gather", case, lambda: lk.experts_gather(x, pair_of, top, rows),
+                  bytes_=pairs * width * 4, like="experts_gather")
+        kb.record("experts gate and up (tensor cores)", case,
+                  lambda: lk.experts_product(rows, up, pair_of, tile_expert, both, False, None,
+                                             ctx.status),
+                  bytes_=2 * weights_read + pairs * (width + 2 * eff) * 2,
+                  tensor_flops=4 * pairs * width * eff, like="experts gate and up")
+        kb.record("clipped_glu", case, lambda: lk.clipped_glu(both, inner, 7.0, 1.702),
+                  bytes_=tiles * seg * eff * 6, like="silu_mul")
+        kb.record("silu_mul (other models)", case, lambda: ops.silu_mul(both, inner),
+                  bytes_=tiles * seg * eff * 6)
+        kb.record("experts down (tensor cores)", case,
+                  lambda: lk.experts_product(inner, down, pair_of, tile_expert, ye, True, None,
+                                             ctx.status),
+                  bytes_=weights_read + pairs * (width + eff) * 2,
+                  tensor_flops=2 * pairs * width * eff, like="experts down")
+        shared = f(n, width).to(bf16)
+        kb.record("experts_combine (with the shared expert)", case,
+                  lambda: lk.experts_combine(ye, weight, eo, None, (shared, side)),
+                  bytes_=n * width * ((top + 1) * 2 + 4), like="experts_combine")
+        kb.record("experts_combine (other models)", case,
+                  lambda: lk.experts_combine(ye, weight, eo), bytes_=n * width * (top * 2 + 4))
+        w_sh, both_s = w(2 * sff, width), torch.empty(n, 2 * sff, dtype=bf16, device=dev)
+        kb.record("linear, the shared expert's gate and up", case,
+                  lambda: ops.linear(x, w_sh, out=both_s, status=ctx.status),
+                  bytes_=(2 * sff * width + n * (width + 2 * sff)) * 2,
+                  tensor_flops=4 * n * width * sff)
+    return kb.rows
+
+
+def workload_puripel(args, warmup: int, steps: int) -> int:
+    """Puripel beside Vapelix (the closest model: latent attention through the same kernels, routed
+    experts), Sebilorn (the closest with states that are carried from token to token) and Llama at
+    equal width, vocabulary and number of layers."""
+    import numpy as np
+    import torch
+    from distengine_b200 import Engine, EngineConfig
+    peak, peak_kind = peaks()
+    layers = args.layers
+    rng = np.random.default_rng(0)
+    vocab = MODEL["vocab_size"]
+    result = {}
+    others = () if args.no_others else (("vapelix", vapelix_folder), ("sebilorn", sebilorn_folder),
+                                        ("llama", model_folder))
+    for name, folder in (("puripel", puripel_folder),) + others:
+        pages = (64 * (PROMPT + 8 + warmup + steps) + PREFILL) // PAGE + 64
+        engine = Engine(folder(layers), EngineConfig(
+            dtype="bfloat16", block_size=PAGE, num_blocks=pages, decode_batch_size=64,
+            max_batch_tokens=PREFILL, max_model_len=4096, use_graphs=not args.no_graphs))
+        entry = {}
+        if args.only != "decode":
+            prefill_ms, prefill_step_ms = timed_prefill(engine, PREFILL, rng, vocab, repeats=5)
+            entry["prefill_2048"] = {"ms": round(prefill_ms, 3),
+                                     "ms_with_host_prepare": round(prefill_step_ms, 3),
+                                     "tokens_per_s": round(PREFILL / prefill_ms * 1e3, 1)}
+        if args.only != "prefill":
+            for batch in (8, 64):
+                ms, launches, _, clocks = timed_decode(engine, batch, PROMPT, steps, warmup, rng,
+                                                       vocab)
+                entry[f"decode_b{batch}"] = {"ms_per_step": round(ms, 4),
+                                             "tokens_per_s": round(batch / ms * 1e3, 1),
+                                             "gpu_launches": int(launches), "clocks": clocks}
+        result[name] = entry
+        del engine
+        torch.cuda.empty_cache()
+    mine = result["puripel"].get("decode_b8", {})
+    print(json.dumps({
+        "metric": "decode tokens/s at batch 8, Puripel at the TinyLlama-1.1B width",
+        "value": mine.get("tokens_per_s"), "unit": "tokens/s", "n_gpus": 1, "steps": steps,
+        "warmup": warmup, "ms_per_step": mine.get("ms_per_step"), "dtype": "bf16",
+        "higher_is_better": True, "data": "synthetic", "impl": "ours", "workload": "puripel",
+        "config": {"layers": layers, "width": MODEL["hidden_size"], "vocab": vocab,
+                   "seq_len": PROMPT, "page_size": PAGE, "peaks": peak_kind,
+                   "shape": puripel_shape(2)["layers"],
+                   "l2": "weights larger than L2 are read every step; kernels alone: L2 flushed"},
+        "gpu_launches": mine.get("gpu_launches"), "clocks": mine.get("clocks"),
+        "models": result, "kernels": [] if args.only != "all" else puripel_kernels(peak)}))
+    return 0
+
+
 def workload_long(args, warmup: int, steps: int) -> int:
     """Llama-3-8B layer sizes: 64 requests with prompts of 4,096 tokens (fed as portions of 4,096
     tokens), then decode steps at batch 64 over the long cache; vocabulary 128,256."""
@@ -1662,9 +2038,12 @@ def main() -> int:
                              "DISTENGINE_B200_DEFINES=DE_TRACE)")
     parser.add_argument("--workload", default="headline",
                         choices=["headline", "mixed", "long", "fp32", "vomotar", "sebilorn",
-                                 "vapelix", "bizetar"])
+                                 "vapelix", "bizetar", "puripel"])
+    parser.add_argument("--no-others", action="store_true",
+                        help="(puripel) without the models it is shown beside")
     args = parser.parse_args()
-    if (args.workload in ("mixed", "long", "vomotar", "sebilorn", "vapelix", "bizetar")
+    if (args.workload in ("mixed", "long", "vomotar", "sebilorn", "vapelix", "bizetar",
+                          "puripel")
             and "--layers" not in " ".join(sys.argv)):
         args.layers = 8          # of the 32 that the Llama-2-7B and Llama-3-8B shapes have
 
@@ -1681,7 +2060,8 @@ def main() -> int:
                 "vomotar": workload_vomotar,
                 "sebilorn": workload_sebilorn,
                 "vapelix": workload_vapelix,
-                "bizetar": workload_bizetar}[args.workload](args, warmup, steps)
+                "bizetar": workload_bizetar,
+                "puripel": workload_puripel}[args.workload](args, warmup, steps)
 
     import numpy as np
     import torch

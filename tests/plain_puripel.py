@@ -279,7 +279,7 @@ def draw(shapes, generator, spread: float = 1.0) -> dict[str, torch.Tensor]:
         if last.startswith("norm"):
             t = 1.0 + 0.2 * r
         elif last == "A_log":
-            t = torch.log(0.5 + 4.0 * torch.rand(shape, generator=g))
+            t = -4.0 + 5.0 * torch.rand(shape, generator=g)
         elif last == "dt_bias":
             t = -3.0 + 1.5 * r
         elif last == "D":
