@@ -1580,6 +1580,7 @@ def puripel_kernels(peak: dict) -> list[dict]:
     from distengine_b200.kernels import ops, ssm
     from distengine_b200.kernels import recurrent as rk
     from distengine_b200.kernels.attention import AttentionLauncher
+    from distengine_b200.parts.context import MixedRows
     from distengine_b200.parts.latent_attention import stretched_frequencies
     from distengine_b200.parts.mamba2 import Mamba2
     dev, bf16 = "cuda:0", torch.bfloat16
@@ -1664,14 +1665,15 @@ def puripel_kernels(peak: dict) -> list[dict]:
             items, portions = ctx.arrays["mamba2/items"], ctx.arrays["mamba2/portions"]
             k = items.shape[0]
             states, decays = torch.empty(k, S, device=dev), torch.empty(k, sz.heads, device=dev)
+            products = torch.empty(k, sz.groups, ssm.CHUNK, ssm.CHUNK, device=dev)
             kb.record("ssm prep (convolution with bias, rates)", case,
                       lambda: ssm.prep(sz, wt, xbc, dt, state, ready, rates, ctx),
                       bytes_=n * C * (2 + 4), like="delta_prep")
 
             def chunks():
-                ssm.chunk_state(sz, ready, rates, items, states, decays)
+                ssm.chunk_state(sz, ready, rates, items, states, decays, products)
                 ssm.chunk_pass(sz, states, decays, portions, state, ctx)
-                ssm.chunk_out(sz, wt, ready, rates, items, states, y)
+                ssm.chunk_out(sz, wt, ready, rates, items, states, products, y)
             # multiply-adds: the state's update and read-out, c . b and the sum over the chunk
             fma = n * (2 * S + sz.groups * ssm.CHUNK * sz.state_dim
                        + sz.heads * ssm.CHUNK * sz.value_dim // 2)
@@ -1679,13 +1681,13 @@ def puripel_kernels(peak: dict) -> list[dict]:
                       bytes_=n * (C + sz.inner) * 4 + 2 * s * S * 4, flops=2 * fma,
                       like="state_scan")
             kb.record("ssm chunk_state", case,
-                      lambda: ssm.chunk_state(sz, ready, rates, items, states, decays),
+                      lambda: ssm.chunk_state(sz, ready, rates, items, states, decays, products),
                       bytes_=n * C * 4 + k * S * 4, flops=2 * n * S)
             kb.record("ssm chunk_pass", case,
                       lambda: ssm.chunk_pass(sz, states, decays, portions, state, ctx),
                       bytes_=2 * k * S * 4)
             kb.record("ssm chunk_out", case,
-                      lambda: ssm.chunk_out(sz, wt, ready, rates, items, states, y),
+                      lambda: ssm.chunk_out(sz, wt, ready, rates, items, states, products, y),
                       bytes_=n * (C + sz.inner) * 4 + k * S * 4, flops=2 * (fma - n * S))
         kb.record("gated_group_norm (kept rows moved on)", case,
                   lambda: ssm.gated_group_norm(y, z, norm_w, mm["norm_groups"], 1e-6, gated, ctx,
@@ -1778,6 +1780,10 @@ def puripel_kernels(peak: dict) -> list[dict]:
                   bytes_=n * width * ((top + 1) * 2 + 4), like="experts_combine")
         kb.record("experts_combine (other models)", case,
                   lambda: lk.experts_combine(ye, weight, eo), bytes_=n * width * (top * 2 + 4))
+        terms = MixedRows(ye, weight, shared, side)
+        kb.record("join_rmsnorm (the experts' sum formed in it)", case,
+                  lambda: ops.join_rmsnorm(resid, terms, norm, None, norm, normed),
+                  bytes_=n * width * ((top + 1) * 2 + 4 + 4 + 2), like="experts_combine")
         w_sh, both_s = w(2 * sff, width), torch.empty(n, 2 * sff, dtype=bf16, device=dev)
         kb.record("linear, the shared expert's gate and up", case,
                   lambda: ops.linear(x, w_sh, out=both_s, status=ctx.status),

@@ -16,6 +16,7 @@
 //                to the state by itself (a matrix product over its tokens), the states at the
 //                chunks' starts one after the other, and every chunk's read-outs:
 //                  y_t = exp(l_t) c_t^T S_start + sum over s <= t of exp(l_t - l_s) dt_s (c_t . b_s) x_s
+//                the products c . b once for all heads of a group;
 //                with l the running sum of a inside the chunk.  The sums l are kept in double
 //                precision: what enters is the difference of two of them, which may be small
 //                between large ones.
@@ -90,45 +91,93 @@ __device__ __forceinline__ float conv_one(const T* __restrict__ xbc, int ld, con
     return silu_f(acc);
 }
 
-// grid (tokens, blocks of channels).  out [n][C], rates [n][2 H]: dt, then a.
-template <typename T, int VEC>
+// The rates of token n, by the block's threads.
+template <typename T>
+__device__ __forceinline__ void rates_of(int n, const T* __restrict__ dt, int ld_dt,
+                                         const float* __restrict__ dt_bias,
+                                         const float* __restrict__ a_log, float* __restrict__ rates,
+                                         int H) {
+    for (int h = threadIdx.x; h < H; h += blockDim.x) {
+        const float d = softplus_f(to_float(dt[(size_t)n * ld_dt + h]) + dt_bias[h]);
+        rates[(size_t)n * 2 * H + h] = d;
+        rates[(size_t)n * 2 * H + H + h] = -expf(a_log[h]) * d;
+    }
+}
+
+// out [n][C], rates [n][2 H]: dt, then a.  grid (runs of RUN tokens, blocks of 512 channels): a
+// thread has four neighbouring channels and keeps their last KK - 1 inputs in registers while it
+// goes through its tokens.  KK = K.
+constexpr int RUN = 8;
+template <typename T, int KK>
+__global__ void __launch_bounds__(128)
+prep_run_kernel(const T* __restrict__ xbc, int ld, const T* __restrict__ dt, int ld_dt, Conv cv,
+                const float* __restrict__ dt_bias, const float* __restrict__ a_log,
+                const int* __restrict__ token_seq, const int* __restrict__ token_slot,
+                const int* __restrict__ positions, const int* __restrict__ seq_pos0,
+                float* __restrict__ out, float* __restrict__ rates, Shape sh, int n_tokens) {
+    const int n0 = blockIdx.x * RUN, n1 = min(n_tokens, n0 + RUN), C = sh.C;
+    const int c = (blockIdx.y * 128 + threadIdx.x) * 4;
+    float w[KK][4], bias[4], x[KK][4];
+    if (c < C) {
+        Quad<float>::load(cv.bias + c, bias);
+#pragma unroll
+        for (int j = 0; j < KK; ++j) Quad<float>::load(cv.taps + (size_t)j * C + c, w[j]);
+    }
+    pdl_wait();
+    if (c < C) {
+        float own[RUN][4];                           // the run's inputs, asked for at once
+#pragma unroll
+        for (int i = 0; i < RUN; ++i)
+            if (n0 + i < n1) Quad<T>::load(xbc + (size_t)(n0 + i) * ld + c, own[i]);
+#pragma unroll
+        for (int i = 0; i < RUN; ++i) {
+            const int n = n0 + i;
+            if (n >= n1) break;
+            const int off = positions[n] - seq_pos0[token_seq[n]];
+            if (i == 0 || off == 0) {                // the inputs before this token
+                const float* kept =
+                    cv.state + (size_t)token_slot[n] * cv.slot_stride + cv.offset;
+#pragma unroll
+                for (int j = 0; j < KK - 1; ++j) {
+                    if (off - (KK - 1) + j >= 0)
+                        Quad<T>::load(xbc + (size_t)(n - (KK - 1) + j) * ld + c, x[j]);
+                    else Quad<float>::load(kept + (size_t)(off + j) * C + c, x[j]);
+                }
+            }
+            float acc[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                x[KK - 1][e] = own[i][e];
+                acc[e] = bias[e];
+#pragma unroll
+                for (int j = 0; j < KK; ++j) acc[e] = fmaf(w[j][e], x[j][e], acc[e]);
+                acc[e] = silu_f(acc[e]);
+#pragma unroll
+                for (int j = 0; j + 1 < KK; ++j) x[j][e] = x[j + 1][e];
+            }
+            Quad<float>::store(out + (size_t)n * C + c, acc);
+        }
+    }
+    if (blockIdx.y == 0)
+        for (int n = n0; n < n1; ++n) rates_of(n, dt, ld_dt, dt_bias, a_log, rates, sh.H);
+    pdl_trigger();
+}
+
+// The same for any K, sizes and alignment: a thread a channel.  grid (tokens, blocks of channels).
+template <typename T>
 __global__ void __launch_bounds__(128)
 prep_kernel(const T* __restrict__ xbc, int ld, const T* __restrict__ dt, int ld_dt, Conv cv,
             const float* __restrict__ dt_bias, const float* __restrict__ a_log,
             const int* __restrict__ token_seq, const int* __restrict__ token_slot,
             const int* __restrict__ positions, const int* __restrict__ seq_pos0,
             float* __restrict__ out, float* __restrict__ rates, Shape sh) {
-    const int n = blockIdx.x, C = sh.C, K = sh.K;
+    const int n = blockIdx.x, C = sh.C;
     const int off = positions[n] - seq_pos0[token_seq[n]];
     const float* kept = cv.state + (size_t)token_slot[n] * cv.slot_stride + cv.offset;
     pdl_wait();
-    const int c = (blockIdx.y * 128 + threadIdx.x) * VEC;
-    if (c < C) {
-        if (VEC == 4) {
-            float acc[4];
-            Quad<float>::load(cv.bias + c, acc);
-            for (int j = 0; j < K; ++j) {
-                const int rel = off - (K - 1) + j;
-                float x[4], w[4];
-                if (rel >= 0) Quad<T>::load(xbc + (size_t)(n - (K - 1) + j) * ld + c, x);
-                else Quad<float>::load(kept + (size_t)(off + j) * C + c, x);
-                Quad<float>::load(cv.taps + (size_t)j * C + c, w);
-#pragma unroll
-                for (int e = 0; e < 4; ++e) acc[e] = fmaf(w[e], x[e], acc[e]);
-            }
-#pragma unroll
-            for (int e = 0; e < 4; ++e) acc[e] = silu_f(acc[e]);
-            Quad<float>::store(out + (size_t)n * C + c, acc);
-        } else {
-            out[(size_t)n * C + c] = conv_one(xbc, ld, cv, kept, n, off, K, C, c);
-        }
-    }
-    if (blockIdx.y == 0)
-        for (int h = threadIdx.x; h < sh.H; h += 128) {
-            const float d = softplus_f(to_float(dt[(size_t)n * ld_dt + h]) + dt_bias[h]);
-            rates[(size_t)n * 2 * sh.H + h] = d;
-            rates[(size_t)n * 2 * sh.H + sh.H + h] = -expf(a_log[h]) * d;
-        }
+    const int c = blockIdx.y * 128 + threadIdx.x;
+    if (c < C) out[(size_t)n * C + c] = conv_one(xbc, ld, cv, kept, n, off, sh.K, C, c);
+    if (blockIdx.y == 0) rates_of(n, dt, ld_dt, dt_bias, a_log, rates, sh.H);
     pdl_trigger();
 }
 
@@ -279,50 +328,106 @@ __device__ __forceinline__ void chunk_sums(const float* __restrict__ rates, int 
     cum[2 * lane + 1] = run;
 }
 
-// rows [count][from .. from + cols) of src into tile [64][pitch], zeros elsewhere; cols <= the
-// tile's columns `width`
-__device__ __forceinline__ void fill_tile(float* tile, int pitch, int width,
-                                          const float* __restrict__ src, size_t ld, int count,
-                                          int cols, int vec) {
+__device__ __forceinline__ void tiles_arrived() {
+    asm volatile("cp.async.wait_all;\n" ::: "memory");
+    __syncthreads();
+}
+
+// The first `count` rows and `cols` columns of src into tile [ROWS][pitch] of WIDTH columns, zeros
+// elsewhere.  The copies are asynchronous: `tiles_arrived` waits for all of them.
+template <int ROWS, int WIDTH>
+__device__ __forceinline__ void fill_tile(float* tile, int pitch, const float* __restrict__ src,
+                                          size_t ld, int count, int cols, int vec) {
     if (vec) {
-        const int quads = width >> 2;
-        for (int i = threadIdx.x; i < L * quads; i += 128) {
-            const int t = i / quads, c = 4 * (i - t * quads);
-            float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-            if (t < count && c < cols) Quad<float>::load(src + t * ld + c, v);
-            Quad<float>::store(tile + t * pitch + c, v);
+        constexpr int QUADS = WIDTH / 4;
+        const unsigned base = (unsigned)__cvta_generic_to_shared(tile);
+#pragma unroll
+        for (int u = 0; u < ROWS * QUADS / 128; ++u) {
+            const int i = threadIdx.x + 128 * u, t = i / QUADS, c = 4 * (i % QUADS);
+            const bool in = t < count && c < cols;   // (outside: no bytes, the rest is zeroed)
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(
+                             base + (unsigned)((t * pitch + c) * sizeof(float))),
+                         "l"(in ? src + t * ld + c : src), "r"(in ? 16 : 0)
+                         : "memory");
         }
     } else {
-        for (int i = threadIdx.x; i < L * width; i += 128) {
-            const int t = i / width, c = i - t * width;
+        for (int i = threadIdx.x; i < ROWS * WIDTH; i += 128) {
+            const int t = i / WIDTH, c = i - t * WIDTH;
             tile[t * pitch + c] = (t < count && c < cols) ? src[t * ld + c] : 0.0f;
         }
     }
 }
 
+// The products c_t . b_s of a chunk's tokens, the same for all heads of a group:
+// products[item][g][t][s] (s <= t is used).  128 threads.
+__device__ __forceinline__ void chunk_products(const float* __restrict__ c_src,
+                                               const float* __restrict__ b_src, const Shape& sh,
+                                               int count, float* Cs, float* Bs,
+                                               float* __restrict__ dst, int vec) {
+    const int tr = threadIdx.x >> 4, tc = threadIdx.x & 15;    // rows tr + 8 i, columns tc + 16 j
+    float G[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) G[i][j] = 0.0f;
+    for (int n0 = 0; n0 < sh.N; n0 += SLICE) {
+        __syncthreads();
+        fill_tile<L, SLICE>(Cs, NARROW, c_src + n0, sh.C, count, min(SLICE, sh.N - n0), vec);
+        fill_tile<L, SLICE>(Bs, NARROW, b_src + n0, sh.C, count, min(SLICE, sh.N - n0), vec);
+        tiles_arrived();
+#pragma unroll 2
+        for (int k = 0; k < SLICE; k += 4) {
+            float b[4][4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) Quad<float>::load(Bs + (tc + 16 * j) * NARROW + k, b[j]);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                float c[4];
+                Quad<float>::load(Cs + (tr + 8 * i) * NARROW + k, c);
+#pragma unroll
+                for (int u = 0; u < 4; ++u)
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) G[i][j] = fmaf(c[u], b[j][u], G[i][j]);
+            }
+        }
+    }
+    pdl_trigger();
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) dst[(tr + 8 * i) * L + tc + 16 * j] = G[i][j];
+}
+
 // What the chunk adds to the state by itself: out[item][h][n][p] = sum_t exp(l_last - l_t) dt_t
-// b_t[n] x_t[p]; decays[item][h] = exp(l_last).  grid (items, H, tiles of n times tiles of p).
-__global__ void __launch_bounds__(128)
+// b_t[n] x_t[p]; decays[item][h] = exp(l_last).  grid (items, H, 1 + tiles of n times tiles of p):
+// of the first layer of blocks one a group forms the products c . b.
+__global__ void __launch_bounds__(128, 6)
 chunk_state_kernel(const float* __restrict__ xbc, const float* __restrict__ rates,
                    const int4* __restrict__ items, float* __restrict__ out,
-                   float* __restrict__ decays, Shape sh, int vec) {
+                   float* __restrict__ decays, float* __restrict__ products, Shape sh, int vec) {
     __shared__ __align__(16) float Bs[L * WIDE], Xs[L * WIDE];
     __shared__ double cum[L];
     __shared__ float dts[L], ws[L];
     const int4 item = items[blockIdx.x];
-    const int h = blockIdx.y, g = h / (sh.H / sh.G), N = sh.N, P = sh.P;
+    const int per = sh.H / sh.G, h = blockIdx.y, g = h / per, N = sh.N, P = sh.P;
     const int p_tiles = (P + 63) >> 6;
-    const int n0 = (blockIdx.z / p_tiles) * 64, p0 = (blockIdx.z % p_tiles) * 64;
     const int tok0 = item.y, count = item.z;
     pdl_wait();
-    chunk_sums(rates, tok0, count, sh.H, h, cum, dts);
     const float* row = xbc + (size_t)tok0 * sh.C;
-    fill_tile(Xs, WIDE, 64, row + h * P + p0, sh.C, count, min(64, P - p0), vec);
-    fill_tile(Bs, WIDE, 64, row + sh.H * P + g * N + n0, sh.C, count, min(64, N - n0), vec);
-    __syncthreads();
+    if (blockIdx.z == 0) {                           // the longest blocks come first
+        if (h % per == 0)
+            chunk_products(row + sh.H * P + (sh.G + g) * N, row + sh.H * P + g * N, sh, count, Bs,
+                           Xs, products + ((size_t)blockIdx.x * sh.G + g) * L * L, vec);
+        return;
+    }
+    const int tile = blockIdx.z - 1, n0 = tile / p_tiles * 64, p0 = tile % p_tiles * 64;
+    fill_tile<L, 64>(Xs, WIDE, row + h * P + p0, sh.C, count, min(64, P - p0), vec);
+    fill_tile<L, 64>(Bs, WIDE, row + sh.H * P + g * N + n0, sh.C, count, min(64, N - n0), vec);
+    chunk_sums(rates, tok0, count, sh.H, h, cum, dts);
+    tiles_arrived();
     if (threadIdx.x < L)
         ws[threadIdx.x] = expf((float)(cum[L - 1] - cum[threadIdx.x])) * dts[threadIdx.x];
-    if (blockIdx.z == 0 && threadIdx.x == 0)
+    if (tile == 0 && threadIdx.x == 0)
         decays[(size_t)blockIdx.x * sh.H + h] = expf((float)cum[L - 1]);
     __syncthreads();
     const int tr = threadIdx.x >> 4, tc = threadIdx.x & 15;     // rows 4 tr, 4 tr + 32; columns 4 tc
@@ -383,7 +488,7 @@ chunk_pass_kernel(float* __restrict__ out, const float* __restrict__ decays,
 #pragma unroll
     for (int e = 0; e < VEC; ++e) S[e] = S_g[e];
     float* chunk = out + (size_t)seq.y * total + at;
-    constexpr int AHEAD = 4;                         // chunks in flight
+    constexpr int AHEAD = 8;                         // chunks in flight
     for (int i0 = 0; i0 < seq.z; i0 += AHEAD) {
         float add[AHEAD][VEC], dec[AHEAD];
 #pragma unroll
@@ -411,61 +516,49 @@ chunk_pass_kernel(float* __restrict__ out, const float* __restrict__ decays,
     for (int e = 0; e < VEC; ++e) S_g[e] = S[e];
 }
 
-// The chunk's read-outs.  grid (items, H, tiles of p).  Thread (tr, tc) has the rows t = tr + 8 i;
-// of the products c . b the columns s = tc + 16 j, of y the columns p = 4 tc + j.
-__global__ void __launch_bounds__(128)
+// The chunk's read-outs.  grid (items, H, tiles of p).  Thread (tr, tc) has the rows t = tr + 8 i
+// and the columns p = 4 tc + j of y.
+__global__ void __launch_bounds__(128, 5)
 chunk_out_kernel(const float* __restrict__ xbc, const float* __restrict__ rates,
                  const int4* __restrict__ items, const float* __restrict__ starts,
-                 const float* __restrict__ skip, float* __restrict__ y, Shape sh, int vec) {
-    // first the stages of c, b [64][NARROW] and the state [SLICE][WIDE]; then x [64][WIDE] where c
-    // and b were
-    __shared__ __align__(16) float stage[2 * L * NARROW], Ss[SLICE * WIDE], Gs[L * WIDE];
+                 const float* __restrict__ products, const float* __restrict__ skip,
+                 float* __restrict__ y, Shape sh, int vec) {
+    // first the stages of c [64][NARROW] and of the state [SLICE][WIDE], then x [64][WIDE]; the
+    // weights of the chunk's tokens beside them
+    __shared__ __align__(16) float stage[L * NARROW + SLICE * WIDE], Gs[L * WIDE];
     __shared__ double cum[L];
     __shared__ float dts[L];
+    static_assert(L * NARROW + SLICE * WIDE >= L * WIDE, "x takes the stages' place");
     const int4 item = items[blockIdx.x];
     const int h = blockIdx.y, g = h / (sh.H / sh.G), N = sh.N, P = sh.P, p0 = blockIdx.z * 64;
     const int tok0 = item.y, count = item.z;
-    float *Cs = stage, *Bs = stage + L * NARROW, *Xs = stage;
+    float *Cs = stage, *Ss = stage + L * NARROW, *Xs = stage;
     const int tr = threadIdx.x >> 4, tc = threadIdx.x & 15;
     pdl_wait();
-    chunk_sums(rates, tok0, count, sh.H, h, cum, dts);
     const float* row = xbc + (size_t)tok0 * sh.C;
-    const float* b_src = row + sh.H * P + g * N;
     const float* c_src = row + sh.H * P + (sh.G + g) * N;
     const float* s_src = starts + ((size_t)blockIdx.x * sh.H + h) * N * P + p0;
     const int p_cols = min(64, P - p0);
-    float G[8][4], Y[8][4];
+    // c . b of the group's chunk, made weights once the running sums are there
+    const float* p_src = products + ((size_t)blockIdx.x * sh.G + g) * L * L;
+    fill_tile<L, 64>(Gs, WIDE, p_src, L, L, L, 1);
+    float Y[8][4];
 #pragma unroll
     for (int i = 0; i < 8; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) G[i][j] = Y[i][j] = 0.0f;
+        for (int j = 0; j < 4; ++j) Y[i][j] = 0.0f;
     for (int n0 = 0; n0 < N; n0 += SLICE) {
         const int cols = min(SLICE, N - n0);
-        __syncthreads();
-        fill_tile(Cs, NARROW, SLICE, c_src + n0, sh.C, count, cols, vec);
-        fill_tile(Bs, NARROW, SLICE, b_src + n0, sh.C, count, cols, vec);
-        if (vec) {
-            for (int i = threadIdx.x; i < SLICE * 16; i += 128) {
-                const int n = i >> 4, p = 4 * (i & 15);
-                float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-                if (n < cols && p < p_cols) Quad<float>::load(s_src + (size_t)(n0 + n) * P + p, v);
-                Quad<float>::store(Ss + n * WIDE + p, v);
-            }
-        } else {
-            for (int i = threadIdx.x; i < SLICE * 64; i += 128) {
-                const int n = i >> 6, p = i & 63;
-                Ss[n * WIDE + p] = (n < cols && p < p_cols) ? s_src[(size_t)(n0 + n) * P + p] : 0.0f;
-            }
-        }
-        __syncthreads();
+        if (n0 > 0) __syncthreads();
+        fill_tile<L, SLICE>(Cs, NARROW, c_src + n0, sh.C, count, cols, vec);
+        fill_tile<SLICE, 64>(Ss, WIDE, s_src + (size_t)n0 * P, P, cols, p_cols, vec);
+        if (n0 == 0) chunk_sums(rates, tok0, count, sh.H, h, cum, dts);
+        tiles_arrived();
 #pragma unroll 2
         for (int k = 0; k < SLICE; k += 4) {
-            float b[4][4], st[4][4];
+            float st[4][4];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                Quad<float>::load(Bs + (tc + 16 * j) * NARROW + k, b[j]);
-                Quad<float>::load(Ss + (k + j) * WIDE + 4 * tc, st[j]);
-            }
+            for (int u = 0; u < 4; ++u) Quad<float>::load(Ss + (k + u) * WIDE + 4 * tc, st[u]);
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
                 float c[4];
@@ -473,28 +566,28 @@ chunk_out_kernel(const float* __restrict__ xbc, const float* __restrict__ rates,
 #pragma unroll
                 for (int u = 0; u < 4; ++u)
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) {
-                        G[i][j] = fmaf(c[u], b[j][u], G[i][j]);
-                        Y[i][j] = fmaf(c[u], st[u][j], Y[i][j]);
-                    }
+                    for (int j = 0; j < 4; ++j) Y[i][j] = fmaf(c[u], st[u][j], Y[i][j]);
             }
         }
     }
     __syncthreads();
-    fill_tile(Xs, WIDE, 64, row + h * P + p0, sh.C, count, p_cols, vec);
+    fill_tile<L, 64>(Xs, WIDE, row + h * P + p0, sh.C, count, p_cols, vec);
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
         const int t = tr + 8 * i;
         const double lt = cum[t];
         const float from_start = expf((float)lt);
+        float m[4];
+        Quad<float>::load(Gs + t * WIDE + 4 * tc, m);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-            const int s = tc + 16 * j;
-            Gs[t * WIDE + s] = s <= t ? G[i][j] * expf((float)(lt - cum[s])) * dts[s] : 0.0f;
+            const int s = 4 * tc + j;
+            m[j] = s <= t ? m[j] * expf((float)(lt - cum[s])) * dts[s] : 0.0f;
             Y[i][j] *= from_start;
         }
+        Quad<float>::store(Gs + t * WIDE + 4 * tc, m);
     }
-    __syncthreads();
+    tiles_arrived();
 #pragma unroll 2
     for (int s = 0; s < L; s += 4) {
         float x[4][4];
@@ -539,13 +632,49 @@ chunk_out_kernel(const float* __restrict__ xbc, const float* __restrict__ rates,
 // ------------------------------------------------------------------------------------------
 struct Keep {
     const void* xbc;
-    int ld, C, K, offset;
+    int ld, C, K, offset, vec;
     float* state;
     long long slot_stride;
     const int *token_seq, *positions, *seq_pos0, *seq_qlen, *seq_slot;
 };
 
-template <typename T, bool VEC>
+// Whether token n is its sequence's last; then the kept inputs move on.  `who` of `of` workers.
+template <typename T>
+__device__ __forceinline__ void keep_inputs(const Keep& kp, int n, int who, int of) {
+    if (kp.K <= 1) return;
+    const int s = kp.token_seq[n], qlen = kp.seq_qlen[s];
+    if (kp.positions[n] - kp.seq_pos0[s] != qlen - 1) return;
+    float* kept = kp.state + (size_t)kp.seq_slot[s] * kp.slot_stride + kp.offset;
+    const T* xbc = (const T*)kp.xbc + (size_t)(n - (qlen - 1)) * kp.ld;
+    constexpr int AT_ONCE = 3;
+    if (kp.K - 1 <= AT_ONCE && kp.vec) {             // all of a quad's new rows, then the stores
+        for (int c = 4 * who; c < kp.C; c += 4 * of) {
+            float v[AT_ONCE][4];
+#pragma unroll
+            for (int i = 0; i < AT_ONCE; ++i) {
+                if (i >= kp.K - 1) break;
+                const int rel = qlen - (kp.K - 1) + i;
+                if (rel >= 0) Quad<T>::load(xbc + (size_t)rel * kp.ld + c, v[i]);
+                else Quad<float>::load(kept + (size_t)(i + qlen) * kp.C + c, v[i]);
+            }
+#pragma unroll
+            for (int i = 0; i < AT_ONCE; ++i) {
+                if (i >= kp.K - 1) break;
+                Quad<float>::store(kept + (size_t)i * kp.C + c, v[i]);
+            }
+        }
+        return;
+    }
+    for (int c = who; c < kp.C; c += of)
+        for (int i = 0; i < kp.K - 1; ++i) {         // ascending: what is read lies ahead
+            const int rel = qlen - (kp.K - 1) + i;
+            kept[(size_t)i * kp.C + c] = rel >= 0 ? to_float(xbc[(size_t)rel * kp.ld + c])
+                                                  : kept[(size_t)(i + qlen) * kp.C + c];
+        }
+}
+
+// A block a (token, part).
+template <typename T>
 __global__ void gated_group_norm_kernel(const float* __restrict__ y, const T* __restrict__ z,
                                         int ldz, const float* __restrict__ weight,
                                         T* __restrict__ out, int cols, int parts, float eps,
@@ -555,53 +684,67 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, const T* __
     const float* yr = y + (size_t)n * cols + base;
     const T* zr = z + (size_t)n * ldz + base;
     pdl_wait();
+    keep_inputs<T>(kp, n, blockIdx.y * blockDim.x + threadIdx.x, gridDim.y * blockDim.x);
     float ss = 0.0f;
-    if (VEC) {
-        for (int i = 4 * threadIdx.x; i < part; i += 4 * blockDim.x) {
-            float a[4], b[4];
-            Quad<float>::load(yr + i, a);
-            Quad<T>::load(zr + i, b);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const float v = a[e] * silu_f(b[e]);
-                ss = fmaf(v, v, ss);
-            }
-        }
-    } else {
-        for (int i = threadIdx.x; i < part; i += blockDim.x) {
-            const float v = yr[i] * silu_f(to_float(zr[i]));
-            ss = fmaf(v, v, ss);
-        }
+    for (int i = threadIdx.x; i < part; i += blockDim.x) {
+        const float v = yr[i] * silu_f(to_float(zr[i]));
+        ss = fmaf(v, v, ss);
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)part + eps);
-    if (VEC) {
-        for (int i = 4 * threadIdx.x; i < part; i += 4 * blockDim.x) {
-            float a[4], b[4], w[4];
-            Quad<float>::load(yr + i, a);
-            Quad<T>::load(zr + i, b);
+    for (int i = threadIdx.x; i < part; i += blockDim.x)
+        out[(size_t)n * cols + base + i] =
+            from_float<T>(yr[i] * silu_f(to_float(zr[i])) * inv * weight[base + i]);
+    pdl_trigger();
+}
+
+// Rows of whole quads, parts of at most 128 QUADS elements: `warps` warps a part, each thread
+// holding QUADS groups of four elements in registers.  A block takes parts of several warps of one
+// token.
+template <typename T, int QUADS>
+__global__ void gated_group_norm_quads_kernel(const float* __restrict__ y, const T* __restrict__ z,
+                                              int ldz, const float* __restrict__ weight,
+                                              T* __restrict__ out, int cols, int parts, int warps,
+                                              float eps, Keep kp) {
+    __shared__ float scratch[32];
+    const int n = blockIdx.x, part = cols / parts, width = 32 * warps;
+    const int mine = blockIdx.y * (blockDim.x / width) + threadIdx.x / width;
+    const int lane = threadIdx.x % width, warp = threadIdx.x >> 5;
+    const size_t base = (size_t)mine * part;
+    const bool live = mine < parts;
+    pdl_wait();
+    keep_inputs<T>(kp, n, blockIdx.y * blockDim.x + threadIdx.x, gridDim.y * blockDim.x);
+    float v[QUADS][4], ss = 0.0f;
+#pragma unroll
+    for (int u = 0; u < QUADS; ++u) {
+        const int i = 4 * (lane + u * width);
+        if (live && i < part) {
+            float b[4];
+            Quad<float>::load(y + (size_t)n * cols + base + i, v[u]);
+            Quad<T>::load(z + (size_t)n * ldz + base + i, b);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                v[u][e] *= silu_f(b[e]);
+                ss = fmaf(v[u][e], v[u][e], ss);
+            }
+        }
+    }
+    ss = warp_sum(ss);
+    if (warps > 1) {
+        if ((threadIdx.x & 31) == 0) scratch[warp] = ss;
+        __syncthreads();
+        ss = 0.0f;
+        for (int u = 0; u < warps; ++u) ss += scratch[warp / warps * warps + u];
+    }
+    const float inv = 1.0f / sqrtf(ss / (float)part + eps);
+#pragma unroll
+    for (int u = 0; u < QUADS; ++u) {
+        const int i = 4 * (lane + u * width);
+        if (live && i < part) {
+            float w[4];
             Quad<float>::load(weight + base + i, w);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) a[e] = a[e] * silu_f(b[e]) * inv * w[e];
-            Quad<T>::store(out + (size_t)n * cols + base + i, a);
-        }
-    } else {
-        for (int i = threadIdx.x; i < part; i += blockDim.x)
-            out[(size_t)n * cols + base + i] =
-                from_float<T>(yr[i] * silu_f(to_float(zr[i])) * inv * weight[base + i]);
-    }
-    if (kp.K > 1) {
-        const int s = kp.token_seq[n], qlen = kp.seq_qlen[s];
-        if (kp.positions[n] - kp.seq_pos0[s] == qlen - 1) {
-            float* kept = kp.state + (size_t)kp.seq_slot[s] * kp.slot_stride + kp.offset;
-            const T* xbc = (const T*)kp.xbc;
-            for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < kp.C;
-                 c += gridDim.y * blockDim.x)
-                for (int i = 0; i < kp.K - 1; ++i) {     // ascending: what is read lies ahead
-                    const int rel = qlen - (kp.K - 1) + i;
-                    kept[(size_t)i * kp.C + c] =
-                        rel >= 0 ? to_float(xbc[(size_t)(n - (qlen - 1) + rel) * kp.ld + c])
-                                 : kept[(size_t)(i + qlen) * kp.C + c];
-                }
+            for (int e = 0; e < 4; ++e) w[e] *= v[u][e] * inv;
+            Quad<T>::store(out + (size_t)n * cols + base + i, w);
         }
     }
     pdl_trigger();
@@ -632,20 +775,33 @@ DE_EXPORT int de_ssm_prep(int dtype, const void* xbc, int ld, const void* dt, in
     const bool vec = sh.C % 4 == 0 && ld % 4 == 0 && aligned16(xbc) && aligned16(taps) &&
                      aligned16(bias) && aligned16(state) && slot_stride % 4 == 0 &&
                      conv_offset % 4 == 0 && aligned16(out);
-    const int per = vec ? 512 : 128;
-    const dim3 grid(n, (sh.C + per - 1) / per);
-    if (grid.y > 65535) return -2;
-#define PREP(T, V)                                                                              \
-    return de_launch(prep_kernel<T, V>, grid, dim3(128), 0, s, (const T*)xbc, ld, (const T*)dt, \
-                     ld_dt, cv, dt_bias, a_log, token_seq, token_slot, positions, seq_pos0, out, \
-                     rates, sh)
-    if (dtype == DE_BF16) {
-        if (vec) PREP(__nv_bfloat16, 4);
-        PREP(__nv_bfloat16, 1);
+#define PREP_ARGS(T)                                                                            \
+    (const T*)xbc, ld, (const T*)dt, ld_dt, cv, dt_bias, a_log, token_seq, token_slot, positions, \
+        seq_pos0, out, rates, sh
+    if (vec && K <= 4) {
+        const dim3 runs((n + RUN - 1) / RUN, (sh.C + 511) / 512);
+        if (runs.y > 65535) return -2;
+#define RUNS(T, KK)                                                                             \
+    return de_launch(prep_run_kernel<T, KK>, runs, dim3(128), 0, s, PREP_ARGS(T), n)
+#define BY_TAPS(T)                                                                              \
+    do {                                                                                        \
+        if (K == 1) RUNS(T, 1);                                                                 \
+        if (K == 2) RUNS(T, 2);                                                                 \
+        if (K == 3) RUNS(T, 3);                                                                 \
+        RUNS(T, 4);                                                                             \
+    } while (0)
+        if (dtype == DE_BF16) BY_TAPS(__nv_bfloat16);
+        BY_TAPS(float);
+#undef BY_TAPS
+#undef RUNS
     }
-    if (vec) PREP(float, 4);
-    PREP(float, 1);
-#undef PREP
+    const dim3 grid(n, (sh.C + 127) / 128);
+    if (grid.y > 65535) return -2;
+    if (dtype == DE_BF16)
+        return de_launch(prep_kernel<__nv_bfloat16>, grid, dim3(128), 0, s,
+                         PREP_ARGS(__nv_bfloat16));
+    return de_launch(prep_kernel<float>, grid, dim3(128), 0, s, PREP_ARGS(float));
+#undef PREP_ARGS
 }
 
 // fused 1: every sequence brings one token; xbc and dt are columns of the projection (type dtype).
@@ -694,14 +850,15 @@ static int chunk_vec(const Shape& sh, const void* a, const void* b) {
 }
 
 DE_EXPORT int de_ssm_chunk_state(const float* xbc, const float* rates, const void* items,
-                                 int n_items, float* out, float* decays, int H, int G, int N,
-                                 int P, int K, void* stream) {
+                                 int n_items, float* out, float* decays, float* products, int H,
+                                 int G, int N, int P, int K, void* stream) {
     if (n_items <= 0) return 0;
     const Shape sh = {H, G, N, P, K, H * P + 2 * G * N};
     if (!shape_ok(sh)) return -2;
-    const dim3 grid(n_items, H, ((N + 63) / 64) * ((P + 63) / 64));
+    const dim3 grid(n_items, H, ((N + 63) / 64) * ((P + 63) / 64) + 1);
+    if (grid.z > 65535) return -2;
     return de_launch(chunk_state_kernel, grid, dim3(128), 0, (cudaStream_t)stream, xbc, rates,
-                     (const int4*)items, out, decays, sh, chunk_vec(sh, xbc, out));
+                     (const int4*)items, out, decays, products, sh, chunk_vec(sh, xbc, out));
 }
 
 DE_EXPORT int de_ssm_chunk_pass(float* out, const float* decays, const void* long_seqs, int n_long,
@@ -722,14 +879,14 @@ DE_EXPORT int de_ssm_chunk_pass(float* out, const float* decays, const void* lon
 }
 
 DE_EXPORT int de_ssm_chunk_out(const float* xbc, const float* rates, const void* items,
-                               int n_items, const float* starts, const float* skip, float* y,
-                               int H, int G, int N, int P, int K, void* stream) {
+                               int n_items, const float* starts, const float* products,
+                               const float* skip, float* y, int H, int G, int N, int P, int K, void* stream) {
     if (n_items <= 0) return 0;
     const Shape sh = {H, G, N, P, K, H * P + 2 * G * N};
     if (!shape_ok(sh)) return -2;
     const dim3 grid(n_items, H, (P + 63) / 64);
     return de_launch(chunk_out_kernel, grid, dim3(128), 0, (cudaStream_t)stream, xbc, rates,
-                     (const int4*)items, starts, skip, y, sh,
+                     (const int4*)items, starts, products, skip, y, sh,
                      chunk_vec(sh, xbc, starts) && aligned16(y));
 }
 
@@ -742,22 +899,38 @@ DE_EXPORT int de_gated_group_norm(int dtype, const float* y, const void* z, int 
                                   const int* seq_qlen, const int* seq_slot, void* stream) {
     if (n <= 0) return 0;
     if (parts <= 0 || cols <= 0 || cols % parts || parts > 65535) return -2;
-    const Keep kp = {xbc, ld_xbc, keep_C, keep_K, keep_offset, state, slot_stride, token_seq,
-                     positions, seq_pos0, seq_qlen, seq_slot};
+    const bool keep_vec = keep_C % 4 == 0 && ld_xbc % 4 == 0 && keep_offset % 4 == 0 &&
+                          slot_stride % 4 == 0 && aligned16(xbc) && aligned16(state);
+    const Keep kp = {xbc, ld_xbc, keep_C, keep_K, keep_offset, keep_vec, state, slot_stride,
+                     token_seq, positions, seq_pos0, seq_qlen, seq_slot};
     cudaStream_t s = (cudaStream_t)stream;
     const int part = cols / parts;
     const bool vec = part % 4 == 0 && ldz % 4 == 0 && aligned16(y) && aligned16(z) &&
                      aligned16(weight) && aligned16(out);
-    const int work = vec ? part / 4 : part;
-    const int threads = work > 256 ? 512 : (work > 128 ? 256 : 128);
-#define NORM(T, V)                                                                              \
-    return de_launch(gated_group_norm_kernel<T, V>, dim3(n, parts), dim3(threads), 0, s, y,     \
-                     (const T*)z, ldz, weight, (T*)out, cols, parts, eps, kp)
-    if (dtype == DE_BF16) {
-        if (vec) NORM(__nv_bfloat16, true);
-        NORM(__nv_bfloat16, false);
+    if (vec && part <= 32 * 32 * 16) {
+        // four quads a thread if the part has them; a power of two of warps, in blocks of at
+        // least 256 threads where there are so many parts
+        int warps = 1;
+        while (warps < 32 && part > 128 * 4 * warps) warps <<= 1;
+        int per = 1;
+        while (per * warps < 8 && per < parts) per <<= 1;
+        const dim3 grid(n, (parts + per - 1) / per), block(32 * warps * per);
+#define NORM(T, Q)                                                                              \
+    return de_launch(gated_group_norm_quads_kernel<T, Q>, grid, block, 0, s, y, (const T*)z,    \
+                     ldz, weight, (T*)out, cols, parts, warps, eps, kp)
+        if (dtype == DE_BF16) {
+            if (part <= 128 * warps) NORM(__nv_bfloat16, 1);
+            NORM(__nv_bfloat16, 4);
+        }
+        if (part <= 128 * warps) NORM(float, 1);
+        NORM(float, 4);
+#undef NORM
     }
-    if (vec) NORM(float, true);
-    NORM(float, false);
+    const int threads = part > 256 ? 512 : (part > 128 ? 256 : 128);
+#define NORM(T)                                                                                 \
+    return de_launch(gated_group_norm_kernel<T>, dim3(n, parts), dim3(threads), 0, s, y,        \
+                     (const T*)z, ldz, weight, (T*)out, cols, parts, eps, kp)
+    if (dtype == DE_BF16) NORM(__nv_bfloat16);
+    NORM(float);
 #undef NORM
 }

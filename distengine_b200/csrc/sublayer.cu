@@ -224,13 +224,55 @@ __global__ void poly_norm_kernel(const T* __restrict__ z, int ldz, const float* 
 // branch joins as it is.  vec null: no vector.  out null: the sum only.  rows: out[i] is the norm
 // of row rows[i], and x stays as it is.  A thread holds CHUNKS groups of four neighbouring elements
 // of the row in registers (CHUNKS 0: the row lies in shared memory, any width).
+// The branch may also come as the terms of a weighted sum (`mixed`): y holds `top` rows for each row
+// of x, summed with weight[row][top], and, unless null, shared[row] times side[row] joins them.
 struct Join {
     const void *wy, *w;
+    const float* weight;       // null: y is the branch's rows
+    const void* shared;        // of y's type
+    const float* side;
+    int top;
     const float* vec;
     const int* rows;
     int width;
     float eps_y, eps;
 };
+
+template <typename Y>
+__device__ __forceinline__ float branch_at(const Y* __restrict__ y, const Join& j, size_t row, int i) {
+    if (j.weight == nullptr) return to_float(y[row * j.width + i]);
+    float s = 0.0f;
+    for (int k = 0; k < j.top; ++k)
+        s = fmaf(j.weight[row * j.top + k], to_float(y[(row * j.top + k) * j.width + i]), s);
+    if (j.shared != nullptr)
+        s = fmaf(j.side[row], to_float(((const Y*)j.shared)[row * j.width + i]), s);
+    return s;
+}
+template <typename Y>
+__device__ __forceinline__ void branch_at4(const Y* __restrict__ y, const Join& j, size_t row, int i,
+                                           float (&b)[4]) {
+    if (j.weight == nullptr) {
+        load4(y + row * j.width + i, b);
+        return;
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) b[e] = 0.0f;
+#pragma unroll 4
+    for (int k = 0; k < j.top; ++k) {
+        const float w = j.weight[row * j.top + k];
+        float t[4];
+        load4(y + (row * j.top + k) * j.width + i, t);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) b[e] = fmaf(w, t[e], b[e]);
+    }
+    if (j.shared != nullptr) {
+        const float w = j.side[row];
+        float t[4];
+        load4((const Y*)j.shared + row * j.width + i, t);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) b[e] = fmaf(w, t[e], b[e]);
+    }
+}
 
 template <typename T, typename Y, typename W, int CHUNKS>
 __global__ void join_rmsnorm_kernel(float* __restrict__ x, const Y* __restrict__ y,
@@ -238,7 +280,6 @@ __global__ void join_rmsnorm_kernel(float* __restrict__ x, const Y* __restrict__
     __shared__ float scratch[33];
     const int row = j.rows ? j.rows[blockIdx.x] : (int)blockIdx.x;
     float* xr = x + (size_t)row * j.width;
-    const Y* yr = y ? y + (size_t)row * j.width : nullptr;
     const W *wy = (const W*)j.wy, *w = (const W*)j.w;
     T* o = out ? out + (size_t)blockIdx.x * j.width : nullptr;
     pdl_wait();
@@ -251,10 +292,10 @@ __global__ void join_rmsnorm_kernel(float* __restrict__ x, const Y* __restrict__
             const int q = threadIdx.x + c * blockDim.x;
             if (q < quads) {
                 load4(xr + 4 * q, v[c]);
-                if (yr) load4(yr + 4 * q, b[c]);
+                if (y) branch_at4(y, j, row, 4 * q, b[c]);
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    if (!yr) b[c][e] = 0.0f;
+                    if (!y) b[c][e] = 0.0f;
                     ss = fmaf(b[c][e], b[c][e], ss);
                 }
             }
@@ -294,17 +335,17 @@ __global__ void join_rmsnorm_kernel(float* __restrict__ x, const Y* __restrict__
     } else {
         extern __shared__ float held[];              // [width]
         float inv = 1.0f, ss = 0.0f;
+        for (int i = threadIdx.x; i < j.width; i += blockDim.x) {
+            const float b = y ? branch_at(y, j, row, i) : 0.0f;
+            held[i] = b;                             // (its own elements only, so no barrier)
+            ss = fmaf(b, b, ss);
+        }
         if (wy) {
-            for (int i = threadIdx.x; i < j.width; i += blockDim.x) {
-                const float b = yr ? to_float(yr[i]) : 0.0f;
-                ss = fmaf(b, b, ss);
-            }
             inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)j.width + j.eps_y);
         }
         ss = 0.0f;
         for (int i = threadIdx.x; i < j.width; i += blockDim.x) {
-            const float b = yr ? to_float(yr[i]) : 0.0f;
-            const float v = xr[i] + b * inv * (wy ? to_float(wy[i]) : 1.0f) +
+            const float v = xr[i] + held[i] * inv * (wy ? to_float(wy[i]) : 1.0f) +
                             (j.vec ? j.vec[i] : 0.0f);
             held[i] = v;
             ss = fmaf(v, v, ss);
@@ -408,18 +449,23 @@ DE_EXPORT int de_poly_norm(int dtype, const void* z, int ldz, const float* coef,
 #undef POLY
 }
 
-// dtype: of out; y_dtype: of y; weight_dtype: of both weights.  n_out: rows of x, or of `rows`.
+// dtype: of out; y_dtype: of y; weight_dtype: of both weights.  mix (with top, shared, side): see
+// Join.  n_out: rows of x, or of `rows`.
 DE_EXPORT int de_join_rmsnorm(int dtype, int y_dtype, int weight_dtype, float* x, const void* y,
+                              const float* mix, int top, const void* shared, const float* side,
                               const void* wy, float eps_y, const float* vec, const void* w,
                               float eps, void* out, const int* rows, int n_out, int width,
                               void* stream) {
     if (n_out <= 0) return 0;
     if (dtype == DE_F32 && y_dtype != DE_F32) return -2;
     cudaStream_t s = (cudaStream_t)stream;
-    const Join j = {wy, w, vec, rows, width, eps_y, eps};
+    if (mix != nullptr && (y == nullptr || top <= 0 || (shared != nullptr && side == nullptr)))
+        return -2;
+    const Join j = {wy, w, mix, shared, side, top, vec, rows, width, eps_y, eps};
     const bool aligned = width % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0 &&
                          (uintptr_t)wy % 16 == 0 && (uintptr_t)vec % 16 == 0 &&
-                         (uintptr_t)w % 16 == 0 && (uintptr_t)out % 16 == 0;
+                         (uintptr_t)w % 16 == 0 && (uintptr_t)out % 16 == 0 &&
+                         (uintptr_t)shared % 16 == 0;
     const int quads = width / 4;
     const size_t smem = (size_t)width * sizeof(float);
     if (smem > 200 * 1024) return -2;

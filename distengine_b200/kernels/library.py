@@ -104,9 +104,9 @@ SIGNATURES: dict[str, dict[str, list]] = {
         "de_ssm_prep": [I, P, I, P, I, P, P, P, P, P, L, I, P, P, P, P, P, P, I, I, I, I, I, I, P],
         "de_ssm_walk": [I, I, P, I, P, I, P, P, P, P, P, P, P, P, L, I, P, P, P, I, I, P, I, I, I,
                         I, I, P],
-        "de_ssm_chunk_state": [P, P, P, I, P, P, I, I, I, I, I, P],
+        "de_ssm_chunk_state": [P, P, P, I, P, P, P, I, I, I, I, I, P],
         "de_ssm_chunk_pass": [P, P, P, I, P, P, L, I, I, I, P],
-        "de_ssm_chunk_out": [P, P, P, I, P, P, P, I, I, I, I, I, P],
+        "de_ssm_chunk_out": [P, P, P, I, P, P, P, P, I, I, I, I, I, P],
         "de_gated_group_norm": [I, P, P, I, P, P, I, I, I, F, P, I, I, I, I, P, L, P, P, P, P, P, P],
     },
     "latent": {
@@ -129,7 +129,7 @@ SIGNATURES: dict[str, dict[str, list]] = {
         "de_gated_normed_add": [I, I, I, P, P, I, P, P, P, P, P, I, I, F, P],
         "de_depth_mix": [I, P, L, P, I, L, P, P, P],
         "de_poly_norm": [I, P, I, P, P, I, I, I, F, P],
-        "de_join_rmsnorm": [I, I, I, P, P, P, F, P, P, F, P, P, I, I, P],
+        "de_join_rmsnorm": [I, I, I, P, P, P, I, P, P, P, F, P, P, F, P, P, I, I, P],
     },
     "attention_decode": {
         "de_attn_decode_head_dim": [], "de_attn_decode_max_cluster": [],

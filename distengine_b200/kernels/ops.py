@@ -296,11 +296,25 @@ def join_rmsnorm(resid: torch.Tensor, y: "torch.Tensor | None", branch_norm=None
                  out: "torch.Tensor | None" = None, rows: "torch.Tensor | None" = None) -> None:
     """resid += y / sqrt(mean(y^2) + eps) * weight + vector row by row in float32, with weight and
     eps of ``branch_norm`` (None: y as it is), y [N, width] (None: no branch) and vector float32
-    [width] (None: none); then, with ``out``, out = the RMS norm ``norm`` of the new rows.
+    [width] (None: none); y may also be the terms of a weighted sum (``parts.context.MixedRows``:
+    ``rows`` [N top, width], ``weight`` [N, top], ``shared``, ``side``).  Then, with ``out``, out = the RMS norm ``norm`` of the new rows.
     ``rows`` (int32): out[i] is the norm of row rows[i], and resid stays as it is."""
     n, width = resid.shape
-    _need(resid.dtype == torch.float32 and resid.is_contiguous() and (y is None or (
-        y.is_contiguous() and y.shape == resid.shape)), "join_rmsnorm: resid float32, y [N, width]")
+    mix = (None, 0, None, None)
+    if y is not None and not isinstance(y, torch.Tensor):
+        weight, shared, side, y = y.weight, y.shared, y.side, y.rows
+        top = weight.shape[1]
+        _need(weight.dtype == torch.float32 and weight.is_contiguous()
+              and weight.shape == (n, top) and y.shape == (n * top, width) and y.is_contiguous()
+              and (shared is None or (
+                  shared.dtype == y.dtype and shared.is_contiguous()
+                  and shared.shape == resid.shape and side.dtype == torch.float32
+                  and side.shape == (n,) and side.is_contiguous())),
+              "join_rmsnorm: rows [N top, width], weight [N, top], shared [N, width], side [N]")
+        mix = (weight.data_ptr(), top, _ptr(shared), _ptr(side) if shared is not None else None)
+    elif y is not None:
+        _need(y.is_contiguous() and y.shape == resid.shape, "join_rmsnorm: y [N, width]")
+    _need(resid.dtype == torch.float32 and resid.is_contiguous(), "join_rmsnorm: resid float32")
     _need(vector is None or (vector.dtype == torch.float32 and vector.is_contiguous()
                              and vector.shape == (width,)), "join_rmsnorm: vector float32 [width]")
     _need((norm is None) == (out is None) and (rows is None or out is not None),
@@ -323,7 +337,7 @@ def join_rmsnorm(resid: torch.Tensor, y: "torch.Tensor | None", branch_norm=None
     lib = library.load("sublayer")
     _check(lib.de_join_rmsnorm(
         _tag(dtype), _tag(y_dtype), _wtag(weights[0]) if weights else 0, resid.data_ptr(), _ptr(y),
-        None if branch_norm is None else branch_norm.weight.data_ptr(),
+        *mix, None if branch_norm is None else branch_norm.weight.data_ptr(),
         0.0 if branch_norm is None else float(branch_norm.eps), _ptr(vector),
         None if norm is None else norm.weight.data_ptr(), 0.0 if norm is None else float(norm.eps),
         _ptr(out), _ptr(rows), n_out, width, _stream()), "join_rmsnorm")

@@ -136,21 +136,28 @@ def walk(sz: Sizes, w: Weights, ready: torch.Tensor, rates: torch.Tensor, state:
                            *sz.tuple(), _stream()), "ssm_walk")
 
 
+def _products(sz: Sizes, products: torch.Tensor, items: int) -> None:
+    _need(products.dtype == torch.float32 and products.is_contiguous()
+          and products.shape == (items, sz.groups, CHUNK, CHUNK),
+          "ssm chunks: products float32 [items, G, CHUNK, CHUNK]")
+
+
 def chunk_state(sz: Sizes, ready: torch.Tensor, rates: torch.Tensor, items: torch.Tensor,
-                states: torch.Tensor, decays: torch.Tensor) -> None:
+                states: torch.Tensor, decays: torch.Tensor, products: torch.Tensor) -> None:
     """What every chunk adds to the state by itself: states [items, state_size] and how much of
-    the state before it is left at its end, decays [items, H].  items int32 [items, 4]: (sequence,
-    first token, tokens, 0)."""
+    the state before it is left at its end, decays [items, H]; and its tokens' c . b, products
+    [items, G, CHUNK, CHUNK].  items int32 [items, 4]: (sequence, first token, tokens, 0)."""
     _rows(sz, ready, rates), _i32(items, "items")
     m = items.shape[0]
     _need(items.shape == (m, 4) and states.dtype == decays.dtype == torch.float32
           and states.is_contiguous() and decays.is_contiguous()
           and states.shape == (m, sz.state_size) and decays.shape == (m, sz.heads),
           "ssm chunks: items [m, 4], states [m, H N P], decays [m, H]")
+    _products(sz, products, m)
     lib = library.load("ssm")
     _check(lib.de_ssm_chunk_state(ready.data_ptr(), rates.data_ptr(), items.data_ptr(), m,
-                                  states.data_ptr(), decays.data_ptr(), *sz.tuple(), _stream()),
-           "ssm_chunk_state")
+                                  states.data_ptr(), decays.data_ptr(), products.data_ptr(),
+                                  *sz.tuple(), _stream()), "ssm_chunk_state")
 
 
 def chunk_pass(sz: Sizes, states: torch.Tensor, decays: torch.Tensor, portions: torch.Tensor,
@@ -166,12 +173,15 @@ def chunk_pass(sz: Sizes, states: torch.Tensor, decays: torch.Tensor, portions: 
 
 
 def chunk_out(sz: Sizes, w: Weights, ready: torch.Tensor, rates: torch.Tensor,
-              items: torch.Tensor, states: torch.Tensor, y: torch.Tensor) -> None:
-    """The read-outs of the chunks' tokens from the states at the chunks' starts."""
+              items: torch.Tensor, states: torch.Tensor, products: torch.Tensor,
+              y: torch.Tensor) -> None:
+    """The read-outs of the chunks' tokens from the states at the chunks' starts and the tokens'
+    c . b."""
+    _products(sz, products, items.shape[0])
     _rows(sz, ready, rates), _results(sz, y, ready.shape[0]), _i32(items, "items")
     lib = library.load("ssm")
     _check(lib.de_ssm_chunk_out(ready.data_ptr(), rates.data_ptr(), items.data_ptr(),
-                                items.shape[0], states.data_ptr(), w.skip.data_ptr(), y.data_ptr(),
+                                items.shape[0], states.data_ptr(), products.data_ptr(), w.skip.data_ptr(), y.data_ptr(),
                                 *sz.tuple(), _stream()), "ssm_chunk_out")
 
 

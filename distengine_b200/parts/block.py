@@ -136,7 +136,10 @@ class SandwichBlock(Block):
         if self.feed_forward is None:
             return
         h = self.feed_forward_norm.forward(stream, ctx)
-        stream.pending = self.feed_forward.forward(h, ctx)
+        if getattr(self.feed_forward, "gives_mixed_rows", False):
+            stream.pending = self.feed_forward.forward(h, ctx, mixed=True)
+        else:
+            stream.pending = self.feed_forward.forward(h, ctx)
         stream.pending_norm = self.feed_forward_after
 
 

@@ -153,6 +153,17 @@ class NormAhead:
         return UnscaledRows(self.rows, self.parts, self.resid.shape[1], self.eps)
 
 
+@dataclass
+class MixedRows:
+    """A branch's output as the terms of a sum that is formed where it joins the stream:
+    row n is sum_k weight[n, k] * rows[n * top + k], plus side[n] * shared[n] where there is one
+    (``weight`` and ``side`` float32, [N, top] and [N])."""
+    rows: torch.Tensor
+    weight: torch.Tensor
+    shared: "torch.Tensor | None" = None
+    side: "torch.Tensor | None" = None
+
+
 class ResidualStream:
     """The residual stream in float32 and the branch output that has not been added yet.
 
@@ -162,7 +173,7 @@ class ResidualStream:
     its result instead of running.
 
     ``pending_norm``: a norm (``weight``, ``eps``) that the pending branch output passes on its way
-    into the stream.  ``pending_vector``: a vector that every row of the stream is still to
+    into the stream (the branch may then be ``MixedRows``).  ``pending_vector``: a vector that every row of the stream is still to
     receive after that.  A norm that cannot fold these calls ``settle`` first."""
 
     def __init__(self, resid: torch.Tensor) -> None:

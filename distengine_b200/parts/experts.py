@@ -35,7 +35,7 @@ import torch
 from ..kernels import latent as lk
 from ..kernels import ops
 from .base import FeedForward, compute_matrix, register_feed_forward
-from .context import StepContext
+from .context import MixedRows, StepContext
 
 
 class RoutedExperts(FeedForward):
@@ -112,7 +112,14 @@ class RoutedExperts(FeedForward):
     def kernel_modules(self):
         return ("experts", "gemm_tcgen05") if self.dtype == torch.bfloat16 else ("experts",)
 
-    def forward(self, x: torch.Tensor, ctx: StepContext, ahead=None) -> torch.Tensor:
+    @property
+    def gives_mixed_rows(self) -> bool:
+        return not self.identity
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, ahead=None,
+                mixed: bool = False) -> "torch.Tensor | MixedRows":
+        """``mixed`` (where ``gives_mixed_rows``): the terms of the weighted sum instead of the sum,
+        for a block that forms it where it joins the stream."""
         n, top = x.shape[0], self.top
         tensor = lk.experts_tensor_ok(x, self.up, n * top, self.down)
         segment = lk.SEGMENT_TENSOR if tensor else lk.SEGMENT
@@ -155,6 +162,8 @@ class RoutedExperts(FeedForward):
             lk.experts_product(inner, self.down, pair_of, tile_expert, y, True, None, ctx.status)
         else:
             lk.experts_down(inner, self.down, pair_of, tile_expert, y)
+        if mixed:
+            return MixedRows(y, weight, *(shared or ()))
         out = ctx.buffer("experts.out", (n, self.width), torch.float32)
         lk.experts_combine(y, weight, out,
                            (chosen, self.experts, x) if self.identity else None, shared)

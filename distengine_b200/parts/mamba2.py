@@ -113,9 +113,11 @@ class Mamba2(ProjectedMixer):
             if items.shape[0]:
                 states = ctx.buffer("mamba2.states", (items.shape[0], s.state_size), f32)
                 decays = ctx.buffer("mamba2.decays", (items.shape[0], s.heads), f32)
-                ssm.chunk_state(s, ready, rates, items, states, decays)
+                products = ctx.buffer("mamba2.products", (items.shape[0], s.groups, ssm.CHUNK,
+                                                          ssm.CHUNK), f32)
+                ssm.chunk_state(s, ready, rates, items, states, decays, products)
                 ssm.chunk_pass(s, states, decays, ctx.arrays["mamba2/portions"], state, ctx)
-                ssm.chunk_out(s, self.weights, ready, rates, items, states, y)
+                ssm.chunk_out(s, self.weights, ready, rates, items, states, products, y)
             if ctx.notes["mamba2"] == 2:
                 ssm.walk(s, self.weights, ready, rates, state, y, ctx)
         gated = ctx.buffer("mamba2.gated", (n, s.inner))

@@ -518,6 +518,32 @@ def test_branch_norm_sum_vector_and_next_norm(dtype, y_dtype, n, width):
         assert_close(resid, new, torch.float32, "the sum alone")
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("n,width,top", [(5, 42, 2), (3, 64, 1), (4, 1024, 5), (2, 9000, 3)])
+def test_a_weighted_sum_is_formed_where_it_joins(dtype, n, width, top):
+    """The experts' outputs and the shared expert's as the terms of a branch: weighted sum, branch
+    norm, stream and next norm in one pass, with and without the shared rows."""
+    from distengine_b200.kernels import ops
+    from distengine_b200.parts.context import MixedRows
+    g = _gen(width + top)
+    x, rows = torch.randn(n, width, generator=g), torch.randn(n * top, width, generator=g).to(dtype)
+    shared, side = torch.randn(n, width, generator=g).to(dtype), torch.rand(n, generator=g)
+    weight = torch.rand(n, top, generator=g)
+    after = _Norm((torch.rand(width, generator=g) + 0.5).to(dtype), 1e-5)
+    before = _Norm((torch.rand(width, generator=g) + 0.5).to(dtype), 1e-6)
+    total = (weight.double()[:, :, None] * rows.double().reshape(n, top, width)).sum(dim=1)
+    for with_shared in (False, True):
+        if with_shared:
+            total = total + side.double()[:, None] * shared.double()
+        extra = (shared.to(DEV), side.to(DEV)) if with_shared else ()
+        resid, out = x.to(DEV).clone(), torch.empty(n, width, dtype=dtype, device=DEV)
+        ops.join_rmsnorm(resid, MixedRows(rows.to(DEV), weight.to(DEV), *extra), after, None,
+                         before, out)
+        new = x.double() + pp.rms_norm(total, after.weight.cpu(), after.eps)
+        assert_close(resid, new, torch.float32, "the stream")
+        assert_close(out, pp.rms_norm(new, before.weight.cpu(), before.eps), dtype, "next norm")
+
+
 @pytest.mark.parametrize("kind", ["rmsnorm", "grouped", "layernorm"])
 def test_norms_fold_what_a_branch_norm_left_pending(kind):
     """A branch with its norm and a vector, read by norms that fold them themselves and by norms
