@@ -189,7 +189,7 @@ prep_kernel(const T* __restrict__ xbc, int ld, const T* __restrict__ dt, int ld_
 // `longest` tokens are walked.
 // ------------------------------------------------------------------------------------------
 template <typename T, bool FUSED, int CQ, int R>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, R <= 8 ? 4 : 2)
 walk_kernel(const T* __restrict__ xbc, int ld, const T* __restrict__ dt_in, int ld_dt, Conv cv,
             const float* __restrict__ dt_bias, const float* __restrict__ a_log,
             const float* __restrict__ ready, const float* __restrict__ rates,
