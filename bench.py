@@ -1613,7 +1613,7 @@ def puripel_kernels(peak: dict) -> list[dict]:
                 adjacent=adjacent), bytes_=n * (H * rot * 4 + 2 * row * 2), like=like)
         mixed = torch.empty(n, H * rank, device=dev)
         sums16 = torch.empty(n, H * row, dtype=bf16, device=dev)
-        for name, size, like in ((f"attention over the latent, window {window}", window,
+        for name, size, like in ((f"attention over the latent, window {window}, exact weights", window,
                                   "attention over the latent"),
                                  ("attention over the latent (other models)", None, "")):
             reach = size or 1 << 30
@@ -1626,7 +1626,8 @@ def puripel_kernels(peak: dict) -> list[dict]:
                     bytes_=read * row * 2 + n * H * (row * 2 + rank * 4),
                     flops=2 * keys * H * (row + rank), like=like)
             else:
-                launcher = AttentionLauncher(bf16, H, 1, row, m["scale"], size)
+                launcher = AttentionLauncher(bf16, H, 1, row, m["scale"], size,
+                                             exact_weights=size is not None)
                 kb.prepare(ctx, lambda prep: launcher.prepare(prep, allow_decode=False))
                 kb.record(name, case, lambda: launcher.run(folded, sums16, pages, pages, table,
                                                            ctx),

@@ -197,7 +197,7 @@ class PuripelConfig(ModelConfig):
                            key_dim=m["dim"], rotary_dim=m["rot_dim"], value_dim=m["vdim"],
                            q_rank=m["q_rank"], kv_rank=m["kv_rank"], scale=m["scale"],
                            theta=m["base"], eps=self.eps, window=m["window"], adjacent=True,
-                           gated=False)
+                           gated=False, exact_weights=True)
 
     def layer_specs(self) -> list[LayerSpec]:
         """A block with a norm before and after each sublayer: windowed latent attention or

@@ -205,7 +205,9 @@ attn_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16
         }
 
         // running softmax
+#if !SPLIT_WEIGHTS
         unsigned pf[RT][NK / 16][4];
+#endif
 #pragma unroll
         for (int rt = 0; rt < RT; ++rt) {
             float m_new[2] = {m_run[2 * rt], m_run[2 * rt + 1]};
@@ -231,8 +233,12 @@ attn_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16
                 const float p3 = fast_exp2((s[rt][j][3] - m_use[1]) * sl);
                 l_add[0] += p0 + p1;
                 l_add[1] += p2 + p3;
+#if SPLIT_WEIGHTS
+                s[rt][j][0] = p0; s[rt][j][1] = p1; s[rt][j][2] = p2; s[rt][j][3] = p3;
+#else
                 pf[rt][j >> 1][(j & 1) * 2] = pack_bf16(p0, p1);
                 pf[rt][j >> 1][(j & 1) * 2 + 1] = pack_bf16(p2, p3);
+#endif
             }
 #pragma unroll
             for (int i = 0; i < 2; ++i)
@@ -247,6 +253,16 @@ attn_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16
         // o += p v
 #pragma unroll
         for (int ks = 0; ks < NK / 16; ++ks) {
+#if SPLIT_WEIGHTS
+            unsigned hi[RT][4], low[RT][4];          // a weight is the sum of its two terms
+#pragma unroll
+            for (int rt = 0; rt < RT; ++rt)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const float* p = &s[rt][2 * ks + (i >> 1)][2 * (i & 1)];
+                    split_bf16(p[0], p[1], hi[rt][i], low[rt][i]);
+                }
+#endif
 #pragma unroll
             for (int jd = 0; jd < DT; jd += 2) {
                 unsigned b[4];
@@ -255,8 +271,15 @@ attn_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16
                                          (jd + (mat >> 1)) * 8);
 #pragma unroll
                 for (int rt = 0; rt < RT; ++rt) {
+#if SPLIT_WEIGHTS
+                    mma_bf16(o_acc[rt][jd], low[rt], b[0], b[1]);
+                    mma_bf16(o_acc[rt][jd + 1], low[rt], b[2], b[3]);
+                    mma_bf16(o_acc[rt][jd], hi[rt], b[0], b[1]);
+                    mma_bf16(o_acc[rt][jd + 1], hi[rt], b[2], b[3]);
+#else
                     mma_bf16(o_acc[rt][jd], pf[rt][ks], b[0], b[1]);
                     mma_bf16(o_acc[rt][jd + 1], pf[rt][ks], b[2], b[3]);
+#endif
                 }
             }
         }

@@ -9,6 +9,12 @@
 #define HEAD_DIM 64
 #endif
 
+// 1: the softmax weights enter their product with the values as two bfloat16 terms instead of one,
+// so that they keep 16 bits of mantissa (attention_mma.cu only)
+#ifndef SPLIT_WEIGHTS
+#define SPLIT_WEIGHTS 0
+#endif
+
 namespace {
 
 constexpr int D = HEAD_DIM;
@@ -59,6 +65,11 @@ __device__ __forceinline__ float fast_exp2(float x) {          // ex2.approx: ex
 __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const unsigned*>(&v);
+}
+// x and y as sums of two bfloat16 numbers each (16 bits of mantissa).
+__device__ __forceinline__ void split_bf16(float x, float y, unsigned& hi, unsigned& low) {
+    hi = pack_bf16(x, y);
+    low = pack_bf16(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
 }
 
 }  // namespace

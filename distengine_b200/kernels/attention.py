@@ -57,7 +57,10 @@ class AttentionLauncher:
 
     def __init__(self, dtype: torch.dtype, heads: int, kv_heads: int, head_dim: int,
                  scale: float, window: "int | None",
-                 device: "torch.device | None" = None) -> None:
+                 device: "torch.device | None" = None, exact_weights: bool = False) -> None:
+        """``exact_weights``: the softmax weights are not rounded to bfloat16 for their product
+        with the values: they enter it as two bfloat16 terms (the mma.sync kernel; steps of single
+        tokens then never take the one-launch kernel)."""
         check_head_dim(head_dim)
         if heads % kv_heads != 0:
             raise ValueError(f"heads ({heads}) must be a multiple of kv_heads ({kv_heads})")
@@ -69,13 +72,14 @@ class AttentionLauncher:
             # wide tiles are 128 rows where the kernel gives a warp two row tiles (head size <= 64)
             self.shapes = [_Shape("wide", 128 if head_dim <= 64 else 64, 0),
                            _Shape("narrow", NARROW_ROWS, 1)]
-            self.module = ("attention_mma", (f"HEAD_DIM={head_dim}",))
+            self.module = ("attention_mma", (f"HEAD_DIM={head_dim}",)
+                           + (("SPLIT_WEIGHTS=1",) if exact_weights else ()))
             self.decode_module = ("attention_decode", (f"HEAD_DIM={head_dim}",))
             # prompt portions at head sizes 64 and 128: the tcgen05 kernel (tensor-memory
             # accumulators, TMA page loads) takes the wide tiles, two row tiles of 128 a block at
             # head size 64 and one at 128; DISTENGINE_B200_ATTENTION=mma keeps the mma.sync one
             self.tcgen05_module = ("attention_tcgen05", (f"HEAD_DIM={head_dim}",))
-            if (head_dim in (64, 128)
+            if (head_dim in (64, 128) and not exact_weights
                     and os.environ.get("DISTENGINE_B200_ATTENTION", "tcgen05") != "mma"):
                 self.shapes[0] = _Shape("wide", 256 if head_dim == 64 else 128, 2)
         else:
@@ -84,13 +88,14 @@ class AttentionLauncher:
         self.fixed_chunk = F32_CHUNK if dtype == torch.float32 else None
         # steps of decoded tokens only: rotation, cache write, attention and merge in one launch;
         # DISTENGINE_B200_DECODE_ATTENTION=split keeps them apart
-        self.fused_decode = (self.tensor_cores and os.environ.get(
+        self.fused_decode = (self.tensor_cores and not exact_weights and os.environ.get(
             "DISTENGINE_B200_DECODE_ATTENTION", "fused") != "split")
         self._decode_blocks_per_sm: "int | None" = None     # asked of the kernel at first use
         self._device = device
         self._sm_count: "int | None" = None                 # asked of the device at first use
         self.key = (f"attention/{'mma' if self.tensor_cores else 'simt'}/{self.group}/"
-                    f"{kv_heads}/{head_dim}/{self.window}")
+                    f"{kv_heads}/{head_dim}/{self.window}"
+                    + ("/exact" if self.tensor_cores and exact_weights else ""))
 
     def _blocks_per_sm(self) -> int:
         """Blocks an SM holds at once: one of the tcgen05 kernel (it takes nearly all shared

@@ -152,8 +152,9 @@ def default_build_requests() -> list[tuple[str, tuple[str, ...]]]:
     requests = [(module, ()) for module in _build.MODULES
                 if module in SIGNATURES
                 and module not in ("attention_mma", "attention_decode", "attention_tcgen05")]
-    # (16: the head size of the tiny model that the smoke test generates with)
+    # (16 and 32: what the tiny models that the smoke test generates with have)
     return (requests + [("attention_mma", (f"HEAD_DIM={d}",)) for d in (16, 64, 128)]
+            + [("attention_mma", ("HEAD_DIM=32", "SPLIT_WEIGHTS=1"))]
             + [("attention_tcgen05", (f"HEAD_DIM={d}",)) for d in (64, 128)]
             + [("attention_decode", (f"HEAD_DIM={d}",)) for d in (16, 64, 128)])
 

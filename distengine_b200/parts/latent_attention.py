@@ -30,7 +30,8 @@ kv_rank features.  Other steps: the CUDA-core kernels of ``csrc/attention_chunk.
 
 Scores, softmax weights, angles and norm statistics are float32; so is the weighted sum over the
 latent on the CUDA-core kernels (the tensor-core kernels round the softmax weights and the sums
-to bfloat16, as they do for every model).
+to bfloat16, as they do for every model; with ``exact_weights`` they take the weights as two
+bfloat16 terms, 16 bits of mantissa).
 """
 
 from __future__ import annotations
@@ -76,7 +77,8 @@ class LatentAttention(Mixer):
     def __init__(self, width: int, heads: int, key_dim: int, rotary_dim: int, value_dim: int,
                  q_rank: int, kv_rank: int, scale: float, theta: float, eps: float,
                  dtype: torch.dtype, device: torch.device, scaling=None,
-                 window: "int | None" = None, adjacent: bool = False, gated: bool = True) -> None:
+                 window: "int | None" = None, adjacent: bool = False, gated: bool = True,
+                 exact_weights: bool = False) -> None:
         super().__init__(dtype, device)
         if window is not None and window <= 0:
             raise ValueError(f"latent_attention: window must be positive or None, got {window}")
@@ -92,12 +94,13 @@ class LatentAttention(Mixer):
         freq, self.magnitude = stretched_frequencies(theta, rotary_dim, scaling)
         self.freq = freq.to(device)
         self.row = kv_rank + rotary_dim              # what a key's row in the pages holds
-        self.key = f"latent_attention/{heads}/{kv_rank}/{rotary_dim}/{window or 0}"
+        self.key = (f"latent_attention/{heads}/{kv_rank}/{rotary_dim}/{window or 0}"
+                    + ("/exact" if exact_weights else ""))
         # prompt portions on the tensor cores: one key/value head of `row` features
         self.launcher = None
         if uses_tensor_cores(dtype, self.row) and self.row <= MAX_HEAD_DIM:
             self.launcher = AttentionLauncher(dtype, heads, 1, self.row, self.scale, window,
-                                              device)
+                                              device, exact_weights)
 
     def tensors(self):
         d, h = self.width, self.heads

@@ -81,7 +81,7 @@ class PagedFixture:
 
 
 def run_paged_attention(fx: PagedFixture, q_list, heads, kv_heads, head_dim, scale, window,
-                        chunk=None, chunks_cap=None, shape=None):
+                        chunk=None, chunks_cap=None, shape=None, exact_weights=False):
     """q_list[i]: [q_len_i, heads, d] float32 queries of the LAST q_len_i positions of sequence i.
     Runs the engine's own launcher (``kernels.attention.AttentionLauncher``): ``chunk`` /
     ``chunks_cap`` pin how key ranges are split (0: not at all, None: the launcher's choice),
@@ -94,7 +94,8 @@ def run_paged_attention(fx: PagedFixture, q_list, heads, kv_heads, head_dim, sca
     qlen = np.array([q.shape[0] for q in q_list], dtype=np.int32)
     pos0 = np.array([n - ql for n, ql in zip(fx.kv_lens, qlen)], dtype=np.int32)
     qstart = (np.cumsum(qlen) - qlen).astype(np.int32)
-    launcher = AttentionLauncher(dtype, heads, kv_heads, head_dim, scale, window)
+    launcher = AttentionLauncher(dtype, heads, kv_heads, head_dim, scale, window,
+                                 exact_weights=exact_weights)
     prep = StepPrep(SimpleNamespace(seq_qlen=qlen, seq_pos0=pos0))
     launcher.prepare(prep, force_chunk=chunk, force_cap=chunks_cap, force_shape=shape,
                      allow_decode=False)

@@ -11,7 +11,7 @@ import torch
 
 import plain_puripel as pp
 import puripel_configs as pc
-from gpu_helpers import PartHarness, assert_close
+from gpu_helpers import PagedFixture, PartHarness, assert_close, run_paged_attention
 
 pytestmark = pytest.mark.gpu
 DEV = "cuda:0"
@@ -60,7 +60,7 @@ def _latent(dtype, width, m, eps):
         "latent_attention", width=width, heads=m["heads"], key_dim=m["dim"],
         rotary_dim=m["rot_dim"], value_dim=m["vdim"], q_rank=m["q_rank"], kv_rank=m["kv_rank"],
         scale=m["scale"], theta=m["rot"]["base"], eps=eps, window=m["mask"]["size"],
-        adjacent=True, gated=False), dtype, torch.device(DEV))
+        adjacent=True, gated=False, exact_weights=True), dtype, torch.device(DEV))
 
 
 def _latent_weights(m, width, seed, spread=1.5):
@@ -75,8 +75,8 @@ LATENT = [
     ((12, 8, 16, 8, 16, 16, 0.3, 17, 10000.0), 4),    # more than 8 heads
     ((1, 32, 4, 1, 8, 60, 0.3, 1, 500.0), 8),         # one head, values of size 1, itself only
     ((5, 4, 32, 24, 40, 8, 0.5, 40, 20.0), 32),       # mostly turned
-    ((6, 24, 16, 20, 32, 48, 0.3, 23, 10000.0), 16),  # cached rows of 64 and of 128 features:
-    ((4, 32, 32, 16, 24, 96, 0.2, 64, 1e6), 16),      # the tcgen05 kernel in bfloat16 prompts
+    ((6, 24, 16, 20, 32, 48, 0.3, 23, 10000.0), 16),  # cached rows of 64 and of 128 features
+    ((4, 32, 32, 16, 24, 96, 0.2, 64, 1e6), 16),
     ((7, 12, 16, 20, 24, 80, 0.3, 2, 10000.0), 4),    # a window of two tokens
     ((4, 8, 8, 8, 8, 16, 0.3, 4096, 10000.0), 16),    # a window beyond everything
 ]
@@ -188,6 +188,33 @@ def test_two_layers_that_differ_in_their_window_only():
         for i, m in enumerate(sizes):
             want = pp.latent_attention(x.double(), _double(ws[i]), "", m, eps, act=_act(dtype))
             assert_close(torch.cat(got[i]), want, dtype, f"window {m['mask']['size']}")
+
+
+@pytest.mark.parametrize("head_dim", [16, 64, 112, 256])
+@pytest.mark.parametrize("window", [40, None])
+@pytest.mark.parametrize("chunk", [0, 64])
+def test_softmax_weights_are_not_rounded_to_sixteen_bits(head_dim, window, chunk):
+    """On the tensor cores with ``exact_weights`` the result is the exact one rounded once, but for
+    elements next to a tie; with weights of one bfloat16 term many more elements differ."""
+    heads, lens, rows = 5, [150, 70], [130, 21]
+    fx = PagedFixture(lens, 1, head_dim, 16, torch.bfloat16, DEV, seed=head_dim)
+    g = _gen(head_dim + chunk)
+    q = [torch.randn(n, heads, head_dim, generator=g).to(torch.bfloat16).float() for n in rows]
+    scale, want = 0.7 / math.sqrt(head_dim), []
+    for i, n in enumerate(rows):
+        at, keys = torch.arange(lens[i] - n, lens[i])[:, None], torch.arange(lens[i])[None, :]
+        seen = (keys <= at) & (at - keys < (window or 1 << 30))
+        s = torch.einsum("ihd,jd->hij", q[i].double(), fx.k[i][:, 0].double()) * scale
+        p = torch.softmax(s.masked_fill(~seen[None], float("-inf")), dim=-1)
+        want.append(torch.einsum("hij,jd->ihd", p, fx.v[i][:, 0].double()).reshape(n, -1))
+    want = torch.cat(want).to(torch.bfloat16).float()
+    unequal = {}
+    for exact in (True, False):
+        got, _ = run_paged_attention(fx, q, heads, 1, head_dim, scale, window, chunk=chunk,
+                                     exact_weights=exact)
+        assert_close(got, want, torch.bfloat16, f"exact {exact}")
+        unequal[exact] = (got != want).float().mean().item()
+    assert unequal[True] < 0.01 < 0.05 < unequal[False], unequal
 
 
 def test_neighbours_are_turned_as_complex_numbers():
