@@ -28,7 +28,8 @@
 // that is linear, r1[h] * (i - j); `sink` [heads], a learned score per head that joins the
 // denominator as exp(sink[h]) without a key or a value (it is added once, when a row's sums are
 // complete, whatever the tiles and the step's cut); and `gate`, sigmoid of which multiplies a
-// row's result in float32 before it is stored (one number a feature or one a head).  qkv_prepare
+// row's result in float32 before it is stored (one number a feature or one a head); `out_scale` is
+// one more factor of every result, for a mixer whose result joins another's.  qkv_prepare
 // is what stands between such a mixer's projection and these kernels (bias, a short convolution
 // over time with the slot's kept rows, norms, rotation, value mixing, the cache write), and
 // conv_keep moves the kept rows on.
@@ -62,6 +63,7 @@ struct Sight {
     const void* gate;   // or null: a row's result is multiplied by sigmoid(gate) before it is
     int ld_gate;        // stored; gate of the queries' type, rows ld_gate apart, one number a
     int gate_per_head;  // feature ([heads dv]) or, with gate_per_head, one a head ([heads])
+    float out_scale;    // every row's result is multiplied by this before it is stored
 };
 template <typename T>
 __device__ __forceinline__ float sight_gate(const Sight& s, size_t token, int head, int dv,
@@ -70,10 +72,10 @@ __device__ __forceinline__ float sight_gate(const Sight& s, size_t token, int he
     const T* g = (const T*)s.gate + token * s.ld_gate + (s.gate_per_head ? head : head * dv + feature);
     return 1.0f / (1.0f + expf(-to_float(*g)));
 }
-// 1 / (the row's sum of weights, with the sink's share): m is the row's reference maximum
+// out_scale / (the row's sum of weights, with the sink's share): m is the row's reference maximum
 __device__ __forceinline__ float sight_inverse(const Sight& s, int head, float m, float l) {
     if (s.sink != nullptr) l += expf(s.sink[head] - m);
-    return l > 0.0f ? 1.0f / l : 0.0f;
+    return l > 0.0f ? s.out_scale / l : 0.0f;
 }
 
 // first key of the near range of a row at `pos` (does not fall as pos grows)
@@ -235,14 +237,17 @@ __global__ void kv_write_rotated_kernel(T* __restrict__ proj, int ld, const int*
 //             step in which every sequence brings one token, so no other block reads the
 //             slot) the block moves the kept rows on itself and conv_keep is not needed
 //   norm      q and k divided by their root mean square (eps inside the root) and weighted: 1 over
-//             every head with weights [dk] that all heads share, 2 over the whole projection with
-//             weights [H dk] and [G dk]
+//             every head with weights [dk] that all heads share (or without weights: a turn keeps
+//             a head's root mean square, so this is also the norm that follows the turn), 2 over
+//             the whole projection with weights [H dk] and [G dk]
 //   freq      the first `rot` features of every head of q and k turned by position, angle = pos *
 //             freq[i] (formed in double precision), cosine and sine times `magnitude`; pairs are
 //             (2i, 2i + 1) with `adjacent`, else (i, i + rot / 2)
 //   temp      q times 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1)
 //   mix       1: the values (as they are cached) are also left in v_first [N, G dv];
 //             2: v <- (1 - lambda) v + lambda v_first, lambda one number on the device
+// With v_from_k the projection has no v columns, C = (H + G) dk, and a head's values are its keys
+// as they stand before the norm and the turn (dv = dk).
 // q goes to q_out [N, H dk] in the activation type, k and v into the pages.  All arithmetic is
 // float32.  One block a token; shared memory: C + rot + H + G floats.
 struct Prepare {
@@ -266,6 +271,7 @@ struct Prepare {
     const float* lambda;
     float* v_first;
     int keep_here;
+    int v_from_k;
 };
 
 // 16 bytes of the projection as floats
@@ -327,7 +333,8 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, T* __rest
     extern __shared__ float sh[];
     __shared__ float scratch[66];
     const int n = blockIdx.x;
-    const int qk = (H + G) * dk, C = qk + G * dv, half = pp.rot / 2;
+    const int qk = (H + G) * dk, C = pp.v_from_k ? qk : qk + G * dv, half = pp.rot / 2;
+    const int v_col = pp.v_from_k ? H * dk : qk;     // where the values stand in sh
     float* cs_tab = sh + C;                          // [half] cosines, then [half] sines
     float* inv_s = cs_tab + pp.rot;                  // [H + G]
     const int pos = positions[n], slot = token_slot[n];
@@ -435,7 +442,8 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, T* __rest
     float temp = 1.0f;
     if (pp.temp_every > 0) temp = 1.0f + pp.temp_coef * logf((float)((pos + 1) / pp.temp_every) + 1.0f);
     const size_t at = ((size_t)(can_write ? page_id : 0) * G) * page + (size_t)(pos % page);
-    const bool paired = dk % 2 == 0 && (pp.adjacent || half == 0);
+    const bool split = !pp.adjacent && half > 0;     // partners half a turned part apart
+    const bool paired = dk % 2 == 0 && (!split || half % 2 == 0);
     // neighbouring features two at a time (turned together, or both plain), one store for both
     for (int idx = threadIdx.x; idx < (paired ? (H + G) * (dk / 2) : 0); idx += blockDim.x) {
         const int h = idx / (dk / 2), i = idx - h * (dk / 2);
@@ -454,7 +462,22 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, T* __rest
                       : k_pages + (at + (size_t)(h - H) * page) * dk;
         const int a = 2 * i, b = a + 1;
         float ra = x[a] * inv * (wt ? wt[a] : 1.0f), rb = x[b] * inv * (wt ? wt[b] : 1.0f);
-        if (i < half) rope_rotate(ra, rb, cs_tab[i], cs_tab[half + i], ra, rb);
+        if (split && a < pp.rot) {                   // both features lie in one half of the turned part
+            const bool first = a < half;
+            const int p = first ? a : a - half, o = first ? a + half : a - half;
+            const float oa = x[o] * inv * (wt ? wt[o] : 1.0f);
+            const float ob = x[o + 1] * inv * (wt ? wt[o + 1] : 1.0f);
+            float other;
+            if (first) {
+                rope_rotate(ra, oa, cs_tab[p], cs_tab[half + p], ra, other);
+                rope_rotate(rb, ob, cs_tab[p + 1], cs_tab[half + p + 1], rb, other);
+            } else {
+                rope_rotate(oa, ra, cs_tab[p], cs_tab[half + p], other, ra);
+                rope_rotate(ob, rb, cs_tab[p + 1], cs_tab[half + p + 1], other, rb);
+            }
+        } else if (!split && i < half) {
+            rope_rotate(ra, rb, cs_tab[i], cs_tab[half + i], ra, rb);
+        }
         store_pair(dst + a, ra * mul, rb * mul);
     }
     const int per = dk - half;                       // work items a head: pairs, then plain features
@@ -485,9 +508,17 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, T* __rest
             dst[a] = from_float<T>(x[a] * inv * (wt ? wt[a] : 1.0f) * mul);
         }
     }
+    if (pp.mix == 0 && dv % 2 == 0) {                // plain values, two at a time
+        for (int idx = threadIdx.x; idx < (can_write ? G * (dv / 2) : 0); idx += blockDim.x) {
+            const int h = idx / (dv / 2), i = 2 * (idx - h * (dv / 2));
+            const float* v = sh + v_col + h * dv + i;
+            store_pair(v_pages + (at + (size_t)h * page) * dv + i, v[0], v[1]);
+        }
+        return;
+    }
     const float lam = pp.mix == 2 ? pp.lambda[0] : 0.0f;
     for (int idx = threadIdx.x; idx < G * dv; idx += blockDim.x) {
-        float v = sh[qk + idx];
+        float v = sh[v_col + idx];
         if (pp.mix == 2) v = (1.0f - lam) * v + lam * pp.v_first[(size_t)n * (G * dv) + idx];
         const T stored = from_float<T>(v);
         if (pp.mix == 1) pp.v_first[(size_t)n * (G * dv) + idx] = to_float(stored);
@@ -1571,13 +1602,13 @@ DE_EXPORT int de_attn_chunk_decode(int dtype, const void* q, int q_stride, void*
                                    const float* fv, int write_kv, const void* gate, int ld_gate,
                                    int v_stride, int linear, const float* sink,
                                    const void* out_gate, int ld_out_gate, int gate_per_head,
-                                   int* status, void* stream) {
+                                   float out_scale, int* status, void* stream) {
     if (n_seqs <= 0) return 0;
     // v_stride 0: values in rows of their own; else rows of v_pages are that many elements apart
     const int pn_v = dtype == DE_BF16 ? 8 : 4;
     if (v_stride != 0 && (v_stride < dv || v_stride % pn_v != 0 || fused)) return -2;
     const Sight sight = {chunk, window, keep_first, softcap, v_stride ? v_stride : dv, linear, sink,
-                         out_gate, ld_out_gate, gate_per_head};
+                         out_gate, ld_out_gate, gate_per_head, out_scale};
     if (out_gate != nullptr && fused) return -2;     // a fused step has its own gate
     const Fuse fuse = {fused, fk, rot, fv, write_kv, gate, ld_gate};
     if (fused && (rot < 0 || rot % 2 || rot > dk || (fv != nullptr && dv % 2) || out_f32)) return -2;
@@ -1663,21 +1694,22 @@ DE_EXPORT int de_qkv_prepare(int dtype, const void* proj, int ld, void* q_out,
                              const float* q_weight, const float* k_weight, float eps,
                              const float* freq, int rot, float magnitude, int adjacent,
                              float temp_coef, int temp_every, int mix, const float* lambda,
-                             float* v_first, int keep_here, int H, int G, int dk, int dv,
-                             void* k_pages, void* v_pages, const int* block_table,
+                             float* v_first, int keep_here, int v_from_k, int H, int G, int dk,
+                             int dv, void* k_pages, void* v_pages, const int* block_table,
                              int table_stride, int page, int num_pages, int n, int* status,
                              void* stream) {
     if (n <= 0) return 0;
     if (rot < 0 || rot % 2 || rot > dk || (rot > 0 && freq == nullptr) || norm < 0 || norm > 2 ||
-        (norm != 0 && (q_weight == nullptr || k_weight == nullptr)) || mix < 0 || mix > 2 ||
+        (norm == 2 && (q_weight == nullptr || k_weight == nullptr)) ||
+        (q_weight == nullptr) != (k_weight == nullptr) || (v_from_k && dv != dk) || mix < 0 || mix > 2 ||
         (mix != 0 && v_first == nullptr) || (mix == 2 && lambda == nullptr) ||
         (taps != nullptr && (K < 1 || (K > 1 && state == nullptr))))
         return -2;
     const Prepare pp = {bias, taps, K, state, slot_stride, conv_offset, norm, q_weight, k_weight,
                         eps, freq, rot, magnitude, adjacent, temp_coef, temp_every, mix, lambda,
-                        v_first, keep_here};
+                        v_first, keep_here, v_from_k};
     cudaStream_t s = (cudaStream_t)stream;
-    const int C = (H + G) * dk + G * dv;
+    const int C = (H + G) * dk + (v_from_k ? 0 : G * dv);
     const size_t smem = (size_t)(C + rot + H + G) * sizeof(float);
     if (smem > 200 * 1024) return -2;
     const int threads = C >= 2048 && n < 512 ? 512 : 256;
@@ -1742,13 +1774,13 @@ DE_EXPORT int de_attn_chunk(int dtype, const void* q, int q_stride, void* out, i
                             int chunk, int window, int keep_first, float softcap, int out_f32,
                             int tile_rows, int v_stride, int linear, const float* sink,
                             const void* out_gate, int ld_out_gate, int gate_per_head,
-                            int* status, void* stream) {
+                            float out_scale, int* status, void* stream) {
     if (num_items <= 0) return 0;
     // v_stride 0: values in rows of their own; else rows of v_pages are that many elements apart
     if (v_stride != 0 && (v_stride < dv || (vec_ok(dtype, dk, dv) && v_stride % (dtype == DE_BF16 ? 8 : 4))))
         return -2;
     const Sight sight = {chunk, window, keep_first, softcap, v_stride ? v_stride : dv, linear, sink,
-                         out_gate, ld_out_gate, gate_per_head};
+                         out_gate, ld_out_gate, gate_per_head, out_scale};
     if (dk <= 0 || dk > MAX_DK || dv <= 0 || dv > MAX_D || heads % kv_heads != 0) return -2;
     cudaStream_t s = (cudaStream_t)stream;
     if (tile_rows != ROWS && !((tile_rows == ROWS * 4 && vec_fits(dtype, dk, dv)) ||

@@ -11,7 +11,8 @@
 //                      square (eps inside the root), powers element by element
 //   join_rmsnorm       x <- x + y / sqrt(mean(y^2) + eps) * w (+ v) and out = the RMS norm of the
 //                      new x: the norm on a branch's result, the sum (with a vector v that every
-//                      row receives) and the norm before the next branch in one pass
+//                      row receives) and the norm before the next branch in one pass; or out =
+//                      the new x rounded, where the next branch reads the stream itself
 //
 // All sums, statistics and the stream are float32 whatever the activation type; every kernel that
 // writes the stream can also write its rounding to the activation type, which the next matrix
@@ -221,7 +222,8 @@ __global__ void poly_norm_kernel(const T* __restrict__ z, int ldz, const float* 
 }
 
 // Y: the branch's type; T: the output's; W: of both norm weights.  y null: no branch.  wy null: the
-// branch joins as it is.  vec null: no vector.  out null: the sum only.  rows: out[i] is the norm
+// branch joins as it is.  vec null: no vector.  out null: the sum only.  w null: out is the sum,
+// rounded.  rows: out[i] is the norm
 // of row rows[i], and x stays as it is.  A thread holds CHUNKS groups of four neighbouring elements
 // of the row in registers (CHUNKS 0: the row lies in shared memory, any width).
 // The branch may also come as the terms of a weighted sum (`mixed`): y holds `top` rows for each row
@@ -319,6 +321,15 @@ __global__ void join_rmsnorm_kernel(float* __restrict__ x, const Y* __restrict__
             }
         }
         if (!o) return;
+        if (!w) {
+            pdl_trigger();
+#pragma unroll
+            for (int c = 0; c < CHUNKS; ++c) {
+                const int q = threadIdx.x + c * blockDim.x;
+                if (q < quads) store4(o + 4 * q, v[c]);
+            }
+            return;
+        }
         inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)j.width + j.eps);
         pdl_trigger();
 #pragma unroll
@@ -352,6 +363,11 @@ __global__ void join_rmsnorm_kernel(float* __restrict__ x, const Y* __restrict__
             if (!j.rows) xr[i] = v;
         }
         if (!o) return;
+        if (!w) {
+            pdl_trigger();
+            for (int i = threadIdx.x; i < j.width; i += blockDim.x) o[i] = from_float<T>(held[i]);
+            return;
+        }
         inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)j.width + j.eps);
         pdl_trigger();
         for (int i = threadIdx.x; i < j.width; i += blockDim.x)

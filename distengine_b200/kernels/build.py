@@ -41,6 +41,7 @@ MODULES: dict[str, tuple[str, tuple[str, ...]]] = {
     "attention_chunk": ("attention_chunk.cu", ()),
     "recurrent": ("recurrent.cu", ()),
     "ssm": ("ssm.cu", ()),
+    "lru": ("lru.cu", ()),
     "latent": ("latent.cu", ()),
     "experts": ("experts.cu", ()),
     "sublayer": ("sublayer.cu", ()),

@@ -76,15 +76,15 @@ SIGNATURES: dict[str, dict[str, list]] = {
         "de_attn_chunk_rows": [I, I, I, I],
         "de_attn_chunk_decode_ok": [I, I, I, I, I, I],
         "de_attn_chunk_decode": [I, P, I, P, I, P, P, P, I, I, P, P, P, I, P, P, I, I, I, I, I, F,
-                                 I, I, I, F, I, I, P, I, P, I, P, I, I, I, P, P, I, I, P, P],
+                                 I, I, I, F, I, I, P, I, P, I, P, I, I, I, P, P, I, I, F, P, P],
         "de_kv_write_rotated": [I, P, I, P, P, P, I, P, I, I, I, I, P, P, P, I, I, I, I, I, P, P],
         "de_attn_finish": [I, P, P, P, P, I, P, I, I, I, I, P],
         "de_conv_keep": [I, P, I, P, L, I, P, P, P, I, I, I, P],
         "de_qkv_prepare": [I, P, I, P, P, P, P, P, P, P, I, P, L, I, I, P, P, F, P, I, F, I, F, I,
-                           I, P, P, I, I, I, I, I, P, P, P, I, I, I, I, P, P],
+                           I, P, P, I, I, I, I, I, I, P, P, P, I, I, I, I, P, P],
         "de_kv_write_normed": [I, P, I, I, P, P, I, I, I, F, P, P, P, I, I, I, I, P, P],
         "de_attn_chunk": [I, P, I, P, I, P, P, P, I, I, P, P, P, P, P, I, P, P, I, I, I, I, I, F,
-                          I, I, I, F, I, I, I, I, P, P, I, I, P, P],
+                          I, I, I, F, I, I, I, I, P, P, I, I, F, P, P],
     },
     "recurrent": {
         "de_recurrent_max_key_dim": [],
@@ -108,6 +108,11 @@ SIGNATURES: dict[str, dict[str, list]] = {
         "de_ssm_chunk_pass": [P, P, P, I, P, P, L, I, I, I, P],
         "de_ssm_chunk_out": [P, P, P, I, P, P, P, P, I, I, I, I, I, P],
         "de_gated_group_norm": [I, P, P, I, P, P, I, I, I, F, P, I, I, I, I, P, L, P, P, P, P, P, P],
+    },
+    "lru": {
+        "de_lru_chunk": [], "de_lru_max_taps": [],
+        "de_lru": [I, I, P, I, P, I, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, P, P, P, P, P, P, I,
+                   F, P, P, P, P],
     },
     "latent": {
         "de_latent_write": [I, I, P, I, P, I, P, I, P, P, P, F, P, F, I, I, I, I, I, P, P, I, I, I,

@@ -297,7 +297,8 @@ def join_rmsnorm(resid: torch.Tensor, y: "torch.Tensor | None", branch_norm=None
     """resid += y / sqrt(mean(y^2) + eps) * weight + vector row by row in float32, with weight and
     eps of ``branch_norm`` (None: y as it is), y [N, width] (None: no branch) and vector float32
     [width] (None: none); y may also be the terms of a weighted sum (``parts.context.MixedRows``:
-    ``rows`` [N top, width], ``weight`` [N, top], ``shared``, ``side``).  Then, with ``out``, out = the RMS norm ``norm`` of the new rows.
+    ``rows`` [N top, width], ``weight`` [N, top], ``shared``, ``side``).  Then, with ``out``, out =
+    the RMS norm ``norm`` of the new rows, or the new rows themselves (rounded) without ``norm``.
     ``rows`` (int32): out[i] is the norm of row rows[i], and resid stays as it is."""
     n, width = resid.shape
     mix = (None, 0, None, None)
@@ -317,8 +318,8 @@ def join_rmsnorm(resid: torch.Tensor, y: "torch.Tensor | None", branch_norm=None
     _need(resid.dtype == torch.float32 and resid.is_contiguous(), "join_rmsnorm: resid float32")
     _need(vector is None or (vector.dtype == torch.float32 and vector.is_contiguous()
                              and vector.shape == (width,)), "join_rmsnorm: vector float32 [width]")
-    _need((norm is None) == (out is None) and (rows is None or out is not None),
-          "join_rmsnorm: a norm and its output come together")
+    _need((norm is None or out is not None) and (rows is None or norm is not None),
+          "join_rmsnorm: a norm has an output, and picked rows a norm")
     if y is None:
         branch_norm = None
     n_out = n

@@ -237,12 +237,12 @@ def mean_of_normed(a: torch.Tensor, b: torch.Tensor, wa: torch.Tensor, wb: torch
 
 # ------------------------------------------------------------------------------- chunk attention
 def _penalty(r1, r2, heads: int, slopes=None, sink=None, gate=None, gate_per_head=False,
-             like=None, value_dim=0):
+             like=None, value_dim=0, out_scale=1.0):
     """The penalty's two pointers and the kernels' last arguments (linear, sink, gate, its row
     stride, whether it is one number a head): either r1 log(1 + r2 distance) or ``slopes``
     [heads] times the distance; ``sink`` [heads]: the softmax's denominator also holds exp(sink);
     ``gate`` [N, heads dv] (or [N, heads] with ``gate_per_head``) of the queries' dtype ``like``:
-    a row's result is multiplied by sigmoid(gate) before it is stored."""
+    a row's result is multiplied by sigmoid(gate) before it is stored, and by ``out_scale``."""
     gated = (None, 0, 0)
     if gate is not None:
         _need(gate.dtype == like and gate.stride(1) == 1 and gate.dim() == 2
@@ -259,8 +259,8 @@ def _penalty(r1, r2, heads: int, slopes=None, sink=None, gate=None, gate_per_hea
             _f32(t, name)
             _need(t.shape == (heads,) and t.is_contiguous(), f"attention: {name} [heads]")
     if slopes is not None:
-        return slopes, slopes, (1, _ptr(sink), *gated)
-    return r1, r2, (0, _ptr(sink), *gated)
+        return slopes, slopes, (1, _ptr(sink), *gated, float(out_scale))
+    return r1, r2, (0, _ptr(sink), *gated, float(out_scale))
 
 
 def chunk_rows_per_tile(dtype: torch.dtype, key_dim: int, value_dim: int, wide: bool,
@@ -307,7 +307,7 @@ def chunk_attention_decode(q: torch.Tensor, out: torch.Tensor, k_pages: torch.Te
                            slopes: "torch.Tensor | None" = None,
                            sink: "torch.Tensor | None" = None,
                            gate: "torch.Tensor | None" = None,
-                           gate_per_head: bool = False) -> None:
+                           gate_per_head: bool = False, out_scale: float = 1.0) -> None:
     """``chunk_attention`` for a step in which every sequence brings one token: a block a
     (sequence, kv head), its warps share the key tiles out; no work items.
 
@@ -325,7 +325,8 @@ def chunk_attention_decode(q: torch.Tensor, out: torch.Tensor, k_pages: torch.Te
           and out.shape[1] == heads * value_dim and q.shape[0] == ctx.n_seqs,
           "chunk_attention_decode: q, out and pages; one token a sequence")
     _i32(block_table, "block_table")
-    r1, r2, last = _penalty(r1, r2, heads, slopes, sink, gate, gate_per_head, q.dtype, value_dim)
+    r1, r2, last = _penalty(r1, r2, heads, slopes, sink, gate, gate_per_head, q.dtype, value_dim,
+                            out_scale)
     extra = (0, None, 0, None, 0, None, 0)
     if fused is not None:
         fk, rot, fv, gate = fused["fk"], fused["rotary_dim"], fused["fv"], fused["gate"]
@@ -390,7 +391,7 @@ def chunk_attention(q: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor,
                     window: int = 0, keep_first: int = 0, softcap: float = 0.0,
                     v_stride: int = 0, slopes: "torch.Tensor | None" = None,
                     sink: "torch.Tensor | None" = None, gate: "torch.Tensor | None" = None,
-                    gate_per_head: bool = False) -> None:
+                    gate_per_head: bool = False, out_scale: float = 1.0) -> None:
     """Attention of the step's rows over the pages: q rows of [heads dk] at the front of ``q``
     (row stride free), out [N, heads dv]; ``tile_rows``: the rows of a tile that ``items`` were
     cut for (``chunk_rows_per_tile``); ``v_stride`` as in ``chunk_attention_decode``; see
@@ -399,7 +400,8 @@ def chunk_attention(q: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor,
           and out.dtype in (q.dtype, torch.float32)
           and out.shape[1] == heads * value_dim, "chunk_attention: q, out and pages")
     _i32(block_table, "block_table"), _i32(items, "items")
-    r1, r2, last = _penalty(r1, r2, heads, slopes, sink, gate, gate_per_head, q.dtype, value_dim)
+    r1, r2, last = _penalty(r1, r2, heads, slopes, sink, gate, gate_per_head, q.dtype, value_dim,
+                            out_scale)
     lib = library.load("attention_chunk")
     _check(lib.de_attn_chunk(_tag(q.dtype), q.data_ptr(), q.stride(0), out.data_ptr(),
                              out.stride(0), k_pages.data_ptr(), v_pages.data_ptr(),
@@ -496,19 +498,22 @@ def qkv_prepare(proj: torch.Tensor, q_out: torch.Tensor, heads: int, kv_heads: i
                 taps: "torch.Tensor | None" = None, kept: "tuple | None" = None,
                 norm: "tuple | None" = None, rotation: "tuple | None" = None,
                 temperature: "tuple | None" = None, mix: "tuple | None" = None,
-                keep_here: bool = False) -> None:
+                keep_here: bool = False, values_from_keys: bool = False) -> None:
     """From the stacked projection ``proj`` = [q (H dk) | k (G dk) | v (G dv) | ...] to the
     queries ``q_out`` [N, H dk] and the keys and values in the pages, through (each optional, in
     this order): ``bias`` float32 [C] (C = (H + G) dk + G dv); ``taps`` float32 [C, K], a causal
     convolution over time whose inputs before the step come from ``kept`` = (state [slots, n],
     offset), laid out as ``conv_keep`` leaves them; ``norm`` = (mode, q weight, k weight, eps),
-    mode "head" (weights [dk]) or "whole" (weights [H dk], [G dk]); ``rotation`` = (freq
+    mode "head" (weights [dk], or both None: no weights) or "whole" (weights [H dk], [G dk]); ``rotation`` = (freq
     [rot / 2], magnitude, adjacent); ``temperature`` = (coef, every) on q; ``mix`` = ("give",
     v_first) or ("take", v_first, lambda [1]) with v_first float32 [N, G dv].  ``keep_here``:
     only for a step in which every sequence brings one token - the kernel then also moves the
-    slots' kept rows on, and no ``conv_keep`` follows."""
+    slots' kept rows on, and no ``conv_keep`` follows.  ``values_from_keys``: there is no v in
+    ``proj`` (C = (H + G) dk, dv = dk): the values are the keys before norm and rotation."""
     n = proj.shape[0]
-    channels = (heads + kv_heads) * key_dim + kv_heads * value_dim
+    channels = (heads + kv_heads) * key_dim + (0 if values_from_keys else kv_heads * value_dim)
+    _need(not values_from_keys or key_dim == value_dim,
+          "qkv_prepare: values that are keys have the keys' size")
     _need(proj.stride(1) == 1 and proj.shape[1] >= channels and proj.dtype == k_pages.dtype
           == v_pages.dtype == q_out.dtype and q_out.is_contiguous()
           and q_out.shape == (n, heads * key_dim), "qkv_prepare: proj, q_out [N, H dk] and pages")
@@ -537,12 +542,13 @@ def qkv_prepare(proj: torch.Tensor, q_out: torch.Tensor, heads: int, kv_heads: i
     if norm is not None:
         mode, qw, kw, eps = norm
         _need(mode in ("head", "whole"), "qkv_prepare: norm over a head or the whole projection")
-        _f32(qw, "q weight"), _f32(kw, "k weight")
-        shapes = ((key_dim,), (key_dim,)) if mode == "head" else ((heads * key_dim,),
-                                                                   (kv_heads * key_dim,))
-        _need((tuple(qw.shape), tuple(kw.shape)) == shapes and qw.is_contiguous()
-              and kw.is_contiguous(), "qkv_prepare: the norm's weights do not fit its mode")
-        normed = (1 if mode == "head" else 2, qw.data_ptr(), kw.data_ptr(), float(eps))
+        if qw is not None or kw is not None or mode == "whole":
+            _f32(qw, "q weight"), _f32(kw, "k weight")
+            shapes = ((key_dim,), (key_dim,)) if mode == "head" else ((heads * key_dim,),
+                                                                       (kv_heads * key_dim,))
+            _need((tuple(qw.shape), tuple(kw.shape)) == shapes and qw.is_contiguous()
+                  and kw.is_contiguous(), "qkv_prepare: the norm's weights do not fit its mode")
+        normed = (1 if mode == "head" else 2, _ptr(qw), _ptr(kw), float(eps))
     turned = (None, 0, 1.0, 0)
     if rotation is not None and rotation[0].numel() > 0:
         freq, magnitude, adjacent = rotation
@@ -567,8 +573,8 @@ def qkv_prepare(proj: torch.Tensor, q_out: torch.Tensor, heads: int, kv_heads: i
     _check(lib.de_qkv_prepare(_tag(proj.dtype), proj.data_ptr(), proj.stride(0), q_out.data_ptr(),
                               ctx.positions.data_ptr(), ctx.token_seq.data_ptr(),
                               ctx.token_slot.data_ptr(), ctx.seq_pos0.data_ptr(), _ptr(bias),
-                              *conv, *normed, *turned, *temp, *mixed, int(bool(keep_here)), heads,
-                              kv_heads, key_dim, value_dim, k_pages.data_ptr(), v_pages.data_ptr(),
+                              *conv, *normed, *turned, *temp, *mixed, int(bool(keep_here)),
+                              int(bool(values_from_keys)), heads, kv_heads, key_dim, value_dim, k_pages.data_ptr(), v_pages.data_ptr(),
                               block_table.data_ptr(), block_table.stride(0), k_pages.shape[2],
                               k_pages.shape[0], n, ctx.status.data_ptr(), _stream()),
            "qkv_prepare")

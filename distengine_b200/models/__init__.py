@@ -1,5 +1,5 @@
-from . import (bizetar, llama, puripel, sebilorn, vapelix,  # noqa: F401  (register the
-               vomotar)                                     # architectures)
+from . import (bizetar, llama, puripel, sebilorn, sifasun,  # noqa: F401  (register the
+               vapelix, vomotar)                            # architectures)
 from .decoder import DecoderModel, expected_tensors
 from .loading import load_model
 

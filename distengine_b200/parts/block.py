@@ -217,6 +217,10 @@ class SublayerNormBlock(Block):
     stream's rounding for the next products (``stream.rows``).  A layer without a feed-forward is
     the first half only.
 
+    Without a gate a sublayer's result stays pending with its norm, and whoever reads the stream
+    next does both in one kernel (``ops.join_rmsnorm``): the next sublayer, which takes the new
+    stream's rounding from it, or the norm behind the last layer.
+
     A sublayer whose only use of its input is one product (it has ``input_matrix()`` and
     ``run(proj, ...)``, as the projected mixers have) shares that product with its gate: the
     gate's matrix is stacked under the sublayer's, so the input is read once and a sublayer
@@ -232,7 +236,10 @@ class SublayerNormBlock(Block):
                                      or not hasattr(norm, "eps") or hasattr(norm, "bias")):
                 raise ValueError("sublayer_norm: the norms on the sublayers' results are RMS "
                                  "norms over the whole row")
+        if depth and not gated:
+            raise ValueError("sublayer_norm: the average over the depth goes with gated sublayers")
         width, dtype, device = mixer_norm.width, mixer.dtype, mixer.device
+        self.gated = gated
         self.mixer_gate = ResidualGate(width, dtype, device) if gated else None
         self.feed_forward_gate = (ResidualGate(width, dtype, device)
                                   if gated and feed_forward is not None else None)
@@ -251,8 +258,6 @@ class SublayerNormBlock(Block):
 
     def _sublayer(self, role, part, gate, h, ctx, cache=None):
         """(the sublayer's result, the gate's product on the same input h)."""
-        if gate is None:
-            raise NotImplementedError("sublayer_norm: only the gated form has a kernel")
         n = h.shape[0]
         if hasattr(part, "input_matrix") and hasattr(part, "run"):
             stack = self._stacks.get(role)
@@ -279,8 +284,37 @@ class SublayerNormBlock(Block):
         None)."""
         ops.gated_normed_add(y, z, gate.bias, norm.weight, norm.eps, stream.resid, out, rows)
 
+    def _read(self, stream: ResidualStream, ctx: StepContext) -> torch.Tensor:
+        """The stream with everything pending in it, rounded to the activation dtype."""
+        resid = stream.resid
+        wide = ctx.dtype == torch.float32
+        if stream.pending is None and stream.pending_vector is None:
+            if wide:
+                return resid
+            if stream.rows is None:
+                stream.rows = ctx.buffer("block.rows", tuple(resid.shape))
+                stream.rows.copy_(resid)
+            return stream.rows
+        rows = None if wide else ctx.buffer("block.rows", tuple(resid.shape))
+        stream.settle(rows)
+        return resid if wide else rows
+
+    def _forward_ungated(self, stream: ResidualStream, ctx: StepContext,
+                         cache: "CacheBinding | None") -> None:
+        if stream.ahead is not None:
+            raise RuntimeError("a block whose sublayers read the stream itself takes no norm that "
+                               "was handed to a product")
+        stream.pending = self.mixer.forward(self._read(stream, ctx), ctx, cache)
+        stream.pending_norm, stream.rows = self.mixer_norm, None
+        if self.feed_forward is not None:
+            stream.pending = self.feed_forward.forward(self._read(stream, ctx), ctx)
+            stream.pending_norm, stream.rows = self.feed_forward_norm, None
+
     def forward(self, stream: ResidualStream, ctx: StepContext, cache: "CacheBinding | None",
                 following=None) -> None:
+        if not self.gated and self.depth_mix is None:
+            self._forward_ungated(stream, ctx, cache)
+            return
         if stream.ahead is not None or stream.pending is not None:
             raise RuntimeError("a block whose sublayers read the stream itself takes a stream "
                                "with nothing pending")

@@ -195,10 +195,12 @@ class ResidualStream:
             self.settle()
         self.pending_vector = vector
 
-    def settle(self) -> None:
-        """Bring everything pending into the stream now."""
+    def settle(self, rows: "torch.Tensor | None" = None) -> None:
+        """Bring everything pending into the stream now.  ``rows`` [N, width] also receives the
+        new stream, rounded to its dtype (and becomes ``self.rows``)."""
         if self.pending is None and self.pending_vector is None:
             return
         from ..kernels import ops
-        ops.join_rmsnorm(self.resid, self.pending, self.pending_norm, self.pending_vector)
+        ops.join_rmsnorm(self.resid, self.pending, self.pending_norm, self.pending_vector, out=rows)
         self.pending = self.pending_norm = self.pending_vector = None
+        self.rows = rows

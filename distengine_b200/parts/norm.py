@@ -6,7 +6,9 @@ the activation dtype, then times the weight.  The block's residual sums
 
 ``groups`` > 1: the row is cut into that many equal consecutive parts and each part is divided by
 its own root mean square; the weight still spans the row.  ``tensor``: the local name of the
-weight (architectures differ in it).
+weight (architectures differ in it).  ``offset`` and ``gain``: what multiplies a row is
+(offset + stored weight) * gain, formed once in float32 when the weight is loaded (a weight stored
+around zero has offset 1; a final norm's gain can hold a factor of the logits).
 
 ``branch_rmsnorm``: the norm on a branch's output before it joins the stream.  It has no kernel of
 its own: the norm that reads the stream next does its work (``ResidualStream.pending_norm``).
@@ -27,18 +29,25 @@ from .context import NormAhead, ResidualStream, StepContext
 
 class RMSNorm(Norm):
     def __init__(self, width: int, eps: float, dtype: torch.dtype, device: torch.device,
-                 groups: int = 1, tensor: str = "weight") -> None:
+                 groups: int = 1, tensor: str = "weight", offset: float = 0.0,
+                 gain: float = 1.0) -> None:
         super().__init__(dtype, device)
         if groups <= 0 or width % groups:
             raise ValueError(f"rmsnorm: groups ({groups}) must divide the width ({width})")
         self.width, self.eps, self.groups, self.tensor = width, eps, groups, tensor
+        self.offset, self.gain = float(offset), float(gain)
         self.weight: "torch.Tensor | None" = None
 
     def tensors(self):
-        return {self.tensor: ((self.width,), "vector")}
+        return {self.tensor: ((self.width,), "bias" if self.offset else "vector")}
 
     def load(self, tensors):
-        self.weight = stored_vector(tensors[self.tensor], self.dtype, self.device)
+        stored = tensors[self.tensor]
+        if self.offset != 0.0 or self.gain != 1.0:
+            self.weight = ((stored.to(torch.float32) + self.offset) * self.gain).to(
+                self.device).contiguous()
+            return
+        self.weight = stored_vector(stored, self.dtype, self.device)
 
     def ahead(self, stream: ResidualStream, ctx: StepContext, count: int):
         if (self.weight.dtype != torch.bfloat16 or stream.pending is not None
@@ -86,8 +95,8 @@ class RMSNorm(Norm):
 
 class BranchNorm(RMSNorm):
     def __init__(self, width: int, eps: float, dtype: torch.dtype, device: torch.device,
-                 tensor: str = "weight") -> None:
-        super().__init__(width, eps, dtype, device, tensor=tensor)
+                 tensor: str = "weight", offset: float = 0.0, gain: float = 1.0) -> None:
+        super().__init__(width, eps, dtype, device, tensor=tensor, offset=offset, gain=gain)
 
     def kernel_modules(self):
         return ("sublayer",)

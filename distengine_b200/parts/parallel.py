@@ -8,6 +8,9 @@ meet:
 
 * ``weighted_sum``: out = scales[0] * branch_0(x) + scales[1] * branch_1(x) with fixed numbers; the
   branches' outputs stay float32 until they are summed.
+* ``joined_sum``: the same sum as one product: what enters the branches' output matrices, times
+  the branch's number (in float32, before it is rounded), stands side by side in one row, and the
+  output matrices stand side by side in one matrix.  For branches with ``run_into``.
 
 The branches are projected mixers (``parts.recurrent.ProjectedMixer``): their input matrices are
 stacked, so the layer's input goes through one product for all of them.  The mixer's cache spec is
@@ -34,9 +37,9 @@ class ParallelMixer(Mixer):
         super().__init__(dtype, device)
         if len(branches) != 2:
             raise ValueError("parallel: two branches side by side are implemented")
-        if combine not in ("mean_of_normed", "weighted_sum"):
+        if combine not in ("mean_of_normed", "weighted_sum", "joined_sum"):
             raise ValueError(f"parallel: combine '{combine}' is not implemented")
-        if combine == "weighted_sum" and (scales is None or len(scales) != 2):
+        if combine != "mean_of_normed" and (scales is None or len(scales) != 2):
             raise ValueError("parallel: a weighted sum needs one scale for each branch")
         self.width, self.eps, self.combine = width, eps, combine
         self.scales = None if scales is None else tuple(float(x) for x in scales)
@@ -45,6 +48,8 @@ class ParallelMixer(Mixer):
         for branch in self.branches:
             if not isinstance(branch, ProjectedMixer):
                 raise ValueError("parallel: a branch must be a projected mixer")
+        if combine == "joined_sum" and any(branch.run_into is None for branch in self.branches):
+            raise ValueError("parallel: a joined sum needs branches with run_into")
         self.graph_safe = all(branch.graph_safe for branch in self.branches)
         self.prepare_key = "parallel/" + "+".join(str(getattr(b, "prepare_key", b.kind))
                                                   for b in self.branches)
@@ -68,6 +73,12 @@ class ParallelMixer(Mixer):
         self.w_in = compute_matrix(stacked, self.dtype, self.device)
         for branch in self.branches:
             branch.finish_load()
+        if self.combine == "joined_sum":
+            # (segments at multiples of 8 columns, zero columns between them)
+            joined, self.out_offsets = stack_segments([b.w_o.t() for b in self.branches])
+            self.w_o = joined.t().contiguous()
+            for branch in self.branches:
+                branch.w_o = None
         if self.combine == "mean_of_normed":
             self.out_weights = [vector32(tensors[f"{name}.out"], self.device)
                                 for name in self.names]
@@ -99,6 +110,18 @@ class ParallelMixer(Mixer):
         proj = ctx.buffer("parallel.proj", (n, self.w_in.shape[0]))
         ops.linear(x, self.w_in, out=proj, status=ctx.status, before=before)
         out = ctx.buffer("parallel.out", (n, self.width))
+        if self.combine == "joined_sum":
+            columns = self.w_o.shape[1]
+            # zero when it is made: the columns between the segments stay so
+            rows_out = ctx.buffer(f"parallel.joined.{columns}." + ".".join(
+                str(b.output_rows()) for b in self.branches), (n, columns), zero=True)
+            for branch, at, rows, to, scale, binding in zip(
+                    self.branches, self.offsets, self.rows, self.out_offsets, self.scales,
+                    cache.parts):
+                branch.run_into(proj[:, at: at + rows], ctx, binding,
+                                rows_out[:, to: to + branch.output_rows()], out_scale=scale)
+            ops.linear(rows_out, self.w_o, out=out, status=ctx.status)
+            return out
         if self.combine == "weighted_sum":
             outs = [branch.run(proj[:, at: at + rows], ctx, binding, out_dtype=torch.float32)
                     for branch, at, rows, binding in zip(self.branches, self.offsets, self.rows,

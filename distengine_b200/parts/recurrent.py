@@ -90,6 +90,11 @@ class ProjectedMixer(Mixer):
             out_dtype: "torch.dtype | None" = None) -> "torch.Tensor | None":
         raise NotImplementedError
 
+    # Optional, for mixers whose output product may be joined with another's: ``output_rows()``,
+    # the columns of ``w_o``, and ``run_into(proj, ctx, cache, out, out_scale)``, which writes what
+    # enters the output product, times a number, into ``out`` [N, output_rows()] (row stride free)
+    run_into = None
+
     def finish_load(self) -> None:
         """Called by whoever owns the input product once the matrix is on the device elsewhere."""
         self._host_in = None
