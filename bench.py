@@ -2,7 +2,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
                     [--workload headline|mixed|long|fp32|vomotar|sebilorn|vapelix|bizetar
-                     |puripel] [--layers L]
+                     |puripel|sifasun] [--layers L]
 
 The default (``headline``) has the TinyLlama-1.1B layer sizes in bfloat16.  A step is one decode
 step of a batch of 8 requests whose prompts of 512 tokens are in the cache; K steps are timed with
@@ -57,6 +57,10 @@ Other workloads, each with its own line (the number of layers is named beside th
   in the others, a norm before and after every sublayer, experts chosen by groups beside a shared
   one) at the same width and vocabulary, beside Vapelix, Sebilorn and Llama with the same number
   of layers, in the same way.
+* ``sifasun``: the Sifasun architecture (windowed attention whose values are the projected keys,
+  alone with a cap and one more term in the softmax's denominator, or beside a gated linear
+  recurrence; norms on the sublayers' results) at the same width and vocabulary, beside Sebilorn,
+  Bizetar and Llama with the same number of layers, in the same way.
 """
 
 from __future__ import annotations
@@ -1793,23 +1797,16 @@ def puripel_kernels(peak: dict) -> list[dict]:
     return kb.rows
 
 
-def workload_puripel(args, warmup: int, steps: int) -> int:
-    """Puripel beside Vapelix (the closest model: latent attention through the same kernels, routed
-    experts), Sebilorn (the closest with states that are carried from token to token) and Llama at
-    equal width, vocabulary and number of layers."""
+def measured_models(args, warmup: int, steps: int, named) -> dict:
+    """Decode at batch 8 and 64 and a prompt of 2,048 tokens of every (name, folder) in turn."""
     import numpy as np
     import torch
     from distengine_b200 import Engine, EngineConfig
-    peak, peak_kind = peaks()
-    layers = args.layers
     rng = np.random.default_rng(0)
-    vocab = MODEL["vocab_size"]
-    result = {}
-    others = () if args.no_others else (("vapelix", vapelix_folder), ("sebilorn", sebilorn_folder),
-                                        ("llama", model_folder))
-    for name, folder in (("puripel", puripel_folder),) + others:
+    vocab, result = MODEL["vocab_size"], {}
+    for name, folder in named:
         pages = (64 * (PROMPT + 8 + warmup + steps) + PREFILL) // PAGE + 64
-        engine = Engine(folder(layers), EngineConfig(
+        engine = Engine(folder(args.layers), EngineConfig(
             dtype="bfloat16", block_size=PAGE, num_blocks=pages, decode_batch_size=64,
             max_batch_tokens=PREFILL, max_model_len=4096, use_graphs=not args.no_graphs))
         entry = {}
@@ -1828,19 +1825,236 @@ def workload_puripel(args, warmup: int, steps: int) -> int:
         result[name] = entry
         del engine
         torch.cuda.empty_cache()
-    mine = result["puripel"].get("decode_b8", {})
+    return result
+
+
+def comparison_line(args, warmup: int, steps: int, name: str, result: dict, shape,
+                    kernels: list) -> int:
+    """Prints the JSON line of a workload that shows model ``name`` beside others."""
+    mine = result[name.lower()].get("decode_b8", {})
     print(json.dumps({
-        "metric": "decode tokens/s at batch 8, Puripel at the TinyLlama-1.1B width",
+        "metric": f"decode tokens/s at batch 8, {name} at the TinyLlama-1.1B width",
         "value": mine.get("tokens_per_s"), "unit": "tokens/s", "n_gpus": 1, "steps": steps,
         "warmup": warmup, "ms_per_step": mine.get("ms_per_step"), "dtype": "bf16",
-        "higher_is_better": True, "data": "synthetic", "impl": "ours", "workload": "puripel",
-        "config": {"layers": layers, "width": MODEL["hidden_size"], "vocab": vocab,
-                   "seq_len": PROMPT, "page_size": PAGE, "peaks": peak_kind,
-                   "shape": puripel_shape(2)["layers"],
+        "higher_is_better": True, "data": "synthetic", "impl": "ours", "workload": name.lower(),
+        "config": {"layers": args.layers, "width": MODEL["hidden_size"],
+                   "vocab": MODEL["vocab_size"], "seq_len": PROMPT, "page_size": PAGE,
+                   "peaks": peaks()[1], "shape": shape,
                    "l2": "weights larger than L2 are read every step; kernels alone: L2 flushed"},
         "gpu_launches": mine.get("gpu_launches"), "clocks": mine.get("clocks"),
-        "models": result, "kernels": [] if args.only != "all" else puripel_kernels(peak)}))
+        "models": result, "kernels": kernels}))
     return 0
+
+
+def workload_puripel(args, warmup: int, steps: int) -> int:
+    """Puripel beside Vapelix (the closest model: latent attention through the same kernels, routed
+    experts), Sebilorn (the closest with states that are carried from token to token) and Llama at
+    equal width, vocabulary and number of layers."""
+    others = () if args.no_others else (("vapelix", vapelix_folder), ("sebilorn", sebilorn_folder),
+                                        ("llama", model_folder))
+    result = measured_models(args, warmup, steps, (("puripel", puripel_folder),) + others)
+    return comparison_line(args, warmup, steps, "Puripel", result, puripel_shape(2)["layers"],
+                           [] if args.only != "all" else puripel_kernels(peaks()[0]))
+
+
+def sifasun_shape(layers: int) -> dict:
+    """A Sifasun model of the headline's width, feed-forward and vocabulary: attention of 16 query
+    heads on 4 key/value heads of 128 features in every layer, in turn alone (window 1,024, a cap)
+    and beside a gated recurrence as wide as the model in 8 parts (window 512, 4 taps).  Every
+    layer has weights of its own."""
+    mlp = {"kind": "dense", "ff": MODEL["intermediate_size"]}
+    common = {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    alone = {"type": "attention", "mlp": mlp,
+             "mixer": dict(common, softcap=30.0, mask={"size": 1024},
+                           rot={"dims": 64, "base": 500000.0, "scaling": {"factor": 8.0}})}
+    beside = {"type": "parallel", "mlp": mlp,
+              "mixer": {"left": dict(common, mask={"size": 512},
+                                     rot={"dims": 128, "base": 10000.0}),
+                        "right": {"width": MODEL["hidden_size"], "blocks": 8, "conv": 4},
+                        "left_scale": 0.5, "right_scale": 0.5}}
+    return {"architecture": "Sifasun", "vocab": MODEL["vocab_size"], "width": MODEL["hidden_size"],
+            "norm": {"eps": 1e-5}, "logit_scale": 1.0,
+            "layers": [[alone, beside][i % 2] for i in range(layers)]}
+
+
+def sifasun_folder(layers: int) -> str:
+    from distengine_b200.weights import write_random_model
+    folder = os.path.join(tempfile.gettempdir(), f"distengine_b200-bench-{os.getuid()}",
+                          f"sifasun-shape-{layers}-layers-seed0-bf16")
+    marker = os.path.join(folder, ".complete")
+    if not os.path.isfile(marker):
+        print("[bench] writing the random-weights model folder ...", file=sys.stderr, flush=True)
+        write_random_model(sifasun_shape(layers), folder, seed=0, dtype="bfloat16",
+                           norm_init="uniform")
+        with open(marker, "w") as handle:
+            handle.write("ok")
+    return folder
+
+
+def sifasun_kernels(peak: dict) -> list[dict]:
+    """The design's kernels alone at the sizes of ``sifasun_shape``, for a prompt of 2,048 tokens
+    and for a decode step of 64 sequences at position 1,500, each beside the like kernel of the
+    other models in the same run (``like``): what prepares q and k (and the values from them)
+    beside Bizetar's preparation, both forms of attention beside Sebilorn's windowed attention and
+    Bizetar's with a sink, the gated recurrence beside the state scan with its preparation
+    (Vomotar's and Sebilorn's) and beside the state-space mixer (Puripel's), the block's row kernel
+    beside the RMS norm."""
+    import torch
+    from types import SimpleNamespace
+    from distengine_b200.kernels import lru, ops, ssm
+    from distengine_b200.kernels import recurrent as rk
+    from distengine_b200.parts.gated_recurrence import GatedRecurrence
+    from distengine_b200.parts.mamba2 import Mamba2
+    from distengine_b200.parts.sink_attention import SinkAttention
+    from distengine_b200.parts.context import CacheBinding
+    dev, bf16 = "cuda:0", torch.bfloat16
+    kb = KernelBench(peak, dev)
+    layers = sifasun_shape(2)["layers"]
+    alone, beside = layers[0]["mixer"], layers[1]["mixer"]
+    width, page = MODEL["hidden_size"], PAGE
+    H, G, d = alone["heads"], alone["kv_heads"], alone["dim"]
+    f = lambda *s: torch.randn(*s, device=dev)
+
+    def attention_part(**more):
+        part = SinkAttention(width, H, G, d, d, d ** -0.5, 1e-5, bf16, torch.device(dev), **more)
+        part.load({name: torch.randn(*shape) if shape else torch.randn(()) for name, (shape, _)
+                   in part.tensors().items()})
+        return part
+
+    for case, lens, pos0 in (("prompt of 2,048", [2048], [0]),
+                             ("decode, 64 sequences", [1] * 64, [1500] * 64)):
+        ctx = kb.context(lens, pos0)
+        n, s = int(sum(lens)), len(lens)
+        longest = max(p + l for p, l in zip(pos0, lens))
+        pages_seq = (longest + page - 1) // page
+        table = torch.arange(s * pages_seq, dtype=torch.int32, device=dev).view(s, pages_seq)
+        kp, vp = (f(s * pages_seq, G, page, d).to(bf16) for _ in range(2))
+        binding = CacheBinding("paged", True, kp, vp, table, page)
+        # ---- what stands between the projection and the attention, then the attention
+        cases = (
+            ("alone: norm a head, window 1024, cap, term of one", dict(
+                norm="head", norm_weighted=False, values_from_keys=True, adjacent=False,
+                rotary_dim=64, frequency_factor=8.0, window=1024, softcap=30.0, sink="zero"),
+             "qkv_prepare", "attention"),
+            ("beside: norm of the projection, window 512", dict(
+                norm="whole", values_from_keys=True, adjacent=False, rotary_dim=128, window=512,
+                sink=None), "qkv_prepare", "attention"),
+            ("other models: norm a head, learned sink (Bizetar)", dict(
+                norm="head", rotary_dim=128, biased=True), "", ""),
+            ("other models: window 1024, cap (Sebilorn)", dict(
+                adjacent=False, rotary_dim=128, window=1024, softcap=30.0, sink=None), "", ""))
+        for name, settings, like_p, like_a in cases:
+            part = attention_part(**settings)
+            if not like_a:
+                part.launcher = None                 # (those models' attention has a gate as well)
+            kb.prepare(ctx, part.prepare)
+            proj = f(n, part.channels).to(bf16)
+            out = torch.empty(n, H * d, dtype=bf16, device=dev)
+            q = torch.empty(n, H * d, dtype=bf16, device=dev)
+            norm = ((part.norm, part.q_norm, part.k_norm, 1e-5) if part.norm else None)
+            kb.record(f"qkv_prepare ({name})", case, lambda: rk.qkv_prepare(
+                proj, q, H, G, d, d, kp, vp, table, ctx, bias=part.bias, norm=norm,
+                rotation=(part.freq, part.magnitude, part.adjacent),
+                values_from_keys=part.values_from_keys),
+                bytes_=n * (part.channels + (H + 2 * G) * d) * 2, like=like_p)
+            reach = part.window or 1 << 30
+            keys = sum(min(p + i + 1, reach) for p, l in zip(pos0, lens) for i in range(l))
+            read = sum(min(p + l, reach + l - 1) for p, l in zip(pos0, lens))
+            kb.record(f"attention ({name})", case,
+                      lambda: part.attend(q, binding, None, out, 1.0, ctx),
+                      bytes_=read * G * d * 4 + n * H * d * 4, like=like_a,
+                      **{"tensor_flops" if part.launcher else "flops": 4 * keys * H * d})
+        # ---- the gated recurrence
+        right = beside["right"]
+        mixer = GatedRecurrence(width, right["width"], right["blocks"], right["conv"], bf16,
+                                torch.device(dev))
+        mixer.load({name: torch.randn(*shape) for name, (shape, _) in mixer.tensors().items()})
+        sz, W = mixer.sizes, right["width"]
+        kb.prepare(ctx, mixer.prepare)
+        proj, out = f(n, 2 * W).to(bf16), torch.empty(n, W, dtype=bf16, device=dev)
+        state = torch.zeros(s, sz.slot_size, device=dev)
+        bind = CacheBinding("state", True, state=state)
+        gate_flops = 4 * n * W * sz.part
+        moved = n * W * (2 + 2 + 2) + 2 * W * sz.part * 2 + s * W * 8
+        if n == s:
+            kb.record("lru step (convolution, gates, state, output branch)", case,
+                      lambda: mixer.run_into(proj, ctx, bind, out),
+                      bytes_=moved + s * W * (sz.taps - 1) * 4 + s * W * 4,
+                      tensor_flops=gate_flops, like="ssm step")
+        else:
+            prod, local = torch.empty(n, W, device=dev), torch.empty(n, W, device=dev)
+            carry = torch.empty(-(-n // lru.CHUNK), W, device=dev)
+            terms = torch.empty(2, n, W, dtype=bf16, device=dev)
+            common = (sz, mixer.weights, proj[:, :W], proj[:, W:], state, out)
+            kb.record("lru (four kernels)", case, lambda: mixer.run_into(proj, ctx, bind, out),
+                      bytes_=moved, tensor_flops=gate_flops, like="ssm chunks")
+            kb.record("lru convolution and gates", case,
+                      lambda: lru.gates(*common, prod, local, ctx, terms),
+                      bytes_=n * W * (2 + 8) + 2 * W * sz.part * 2, tensor_flops=gate_flops)
+            kb.record("lru carry", case, lambda: lru.carry_on(*common, prod, local, carry, ctx),
+                      bytes_=carry.numel() * 12)
+            kb.record("lru out", case, lambda: lru.finish(*common, prod, local, carry, ctx),
+                      bytes_=n * W * (8 + 2 + 2))
+        # ---- other models' kernels that carry a state
+        m2 = ssm.Sizes(64, 8, 128, 64, 4)
+        C, S = m2.channels, m2.state_size
+        wt = ssm.Weights(f(m2.taps, C), f(C), f(m2.heads) - 2, f(m2.heads), f(m2.heads))
+        mproj = f(n, m2.inner + C + m2.heads).to(bf16)
+        _, xbc, dt = mproj.split([m2.inner, C, m2.heads], dim=1)
+        mstate, y = torch.zeros(s, m2.slot_size, device=dev), torch.empty(n, m2.inner, device=dev)
+        mmoved = n * (C * 2 + m2.inner * 4) + 2 * s * S * 4
+        if n == s:
+            kb.record("ssm step (other models: Puripel)", case,
+                      lambda: ssm.step(m2, wt, xbc, dt, mstate, y, ctx),
+                      bytes_=mmoved + n * (m2.taps - 1) * C * 4, flops=5 * n * S)
+        else:
+            ssm_mixer = Mamba2(width, 64, 8, 128, 64, 4, 8, 1e-6, bf16, torch.device(dev))
+            kb.prepare(ctx, ssm_mixer.prepare)
+            ready, rates = torch.empty(n, C, device=dev), torch.empty(n, 2 * m2.heads, device=dev)
+            items, portions = ctx.arrays["mamba2/items"], ctx.arrays["mamba2/portions"]
+            k = items.shape[0]
+            states, decays = torch.empty(k, S, device=dev), torch.empty(k, m2.heads, device=dev)
+            products = torch.empty(k, m2.groups, ssm.CHUNK, ssm.CHUNK, device=dev)
+
+            def chunks():
+                ssm.prep(m2, wt, xbc, dt, mstate, ready, rates, ctx)
+                ssm.chunk_state(m2, ready, rates, items, states, decays, products)
+                ssm.chunk_pass(m2, states, decays, portions, mstate, ctx)
+                ssm.chunk_out(m2, wt, ready, rates, items, states, products, y)
+            fma = n * (2 * S + m2.groups * ssm.CHUNK * m2.state_dim
+                       + m2.heads * ssm.CHUNK * m2.value_dim // 2)
+            kb.record("ssm prep and chunks (other models: Puripel)", case, chunks,
+                      bytes_=n * (C + m2.inner) * 4 + 2 * s * S * 4, flops=2 * fma)
+        dh, dd = 16, 128
+        qn, kn, vv = f(n, dh * dd), f(n, dh * dd), f(n, dh * dd)
+        decay, o = torch.rand(dh, device=dev), torch.empty(n, dh * dd, device=dev)
+        sstate = torch.zeros(s, dh * dd * dd, device=dev)
+        kb.record("state_scan (other models: retention)", case,
+                  lambda: rk.state_scan(qn, kn, vv, sstate, o, dh, dh, dd, dd, ctx, decay=decay),
+                  bytes_=2 * s * dh * dd * dd * 4 + n * dh * dd * 16, flops=n * dh * dd * dd * 5)
+        # ---- the norm on a sublayer's result
+        resid, branch = f(n, width), f(n, width).to(bf16)
+        norm = SimpleNamespace(weight=torch.rand(width, device=dev), eps=1e-5)
+        rows = torch.empty(n, width, dtype=bf16, device=dev)
+        kb.record("join_rmsnorm (branch norm, sum, rounding)", case,
+                  lambda: ops.join_rmsnorm(resid, branch, norm, out=rows),
+                  bytes_=n * width * (4 + 4 + 2 + 2), like="add_rmsnorm")
+        weight = norm.weight.to(bf16)
+        kb.record("add_rmsnorm (other models)", case,
+                  lambda: ops.add_rmsnorm(resid, branch, weight, 1e-5, rows),
+                  bytes_=n * width * (4 + 4 + 2 + 2))
+    return kb.rows
+
+
+def workload_sifasun(args, warmup: int, steps: int) -> int:
+    """Sifasun beside Sebilorn (the closest model: windowed attention with a cap, and attention
+    beside a recurrence), Bizetar (attention with a sink, norms on the sublayers' results) and
+    Llama at equal width, vocabulary and number of layers."""
+    others = () if args.no_others else (("sebilorn", sebilorn_folder), ("bizetar", bizetar_folder),
+                                        ("llama", model_folder))
+    result = measured_models(args, warmup, steps, (("sifasun", sifasun_folder),) + others)
+    return comparison_line(args, warmup, steps, "Sifasun", result, sifasun_shape(2)["layers"],
+                           [] if args.only != "all" else sifasun_kernels(peaks()[0]))
 
 
 def workload_long(args, warmup: int, steps: int) -> int:
@@ -2045,12 +2259,12 @@ def main() -> int:
                              "DISTENGINE_B200_DEFINES=DE_TRACE)")
     parser.add_argument("--workload", default="headline",
                         choices=["headline", "mixed", "long", "fp32", "vomotar", "sebilorn",
-                                 "vapelix", "bizetar", "puripel"])
+                                 "vapelix", "bizetar", "puripel", "sifasun"])
     parser.add_argument("--no-others", action="store_true",
-                        help="(puripel) without the models it is shown beside")
+                        help="(puripel, sifasun) without the models it is shown beside")
     args = parser.parse_args()
     if (args.workload in ("mixed", "long", "vomotar", "sebilorn", "vapelix", "bizetar",
-                          "puripel")
+                          "puripel", "sifasun")
             and "--layers" not in " ".join(sys.argv)):
         args.layers = 8          # of the 32 that the Llama-2-7B and Llama-3-8B shapes have
 
@@ -2068,7 +2282,8 @@ def main() -> int:
                 "sebilorn": workload_sebilorn,
                 "vapelix": workload_vapelix,
                 "bizetar": workload_bizetar,
-                "puripel": workload_puripel}[args.workload](args, warmup, steps)
+                "puripel": workload_puripel,
+                "sifasun": workload_sifasun}[args.workload](args, warmup, steps)
 
     import numpy as np
     import torch

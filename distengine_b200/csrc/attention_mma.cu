@@ -16,6 +16,10 @@
 // as in src/layers/attention.py:41-64 plus an optional window.  An item that covers a chunk of a
 // long key range writes an unnormalised partial (accumulator, maximum, sum) in the layout that
 // `de_attn_combine` merges.
+// Built with -DSCORE_EXTRAS=1 the kernel also takes a soft cap on the scores, score <- cap *
+// tanh(score / cap); a sink, one number per head whose exponential joins the denominator without a
+// key or a value (of a key range that is cut, the first chunk's partial holds it); and a factor of
+// every result.
 
 #include "common.cuh"
 
@@ -38,7 +42,8 @@ attn_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16
                 const int* __restrict__ seq_qstart, const int* __restrict__ seq_qlen,
                 const int* __restrict__ seq_pos0, const WorkItem* __restrict__ items,
                 float* __restrict__ partial_acc, float* __restrict__ partial_ml, int heads,
-                int kv_heads, int page, float scale, int window, int* __restrict__ status) {
+                int kv_heads, int page, float scale, int window, float softcap,
+                const float* __restrict__ sink, float out_scale, int* __restrict__ status) {
     static_assert(WN == 1 || RT == 1, "warps that split the keys own one row tile");
     constexpr int ROWS = WM * 16 * RT;     // rows of the tile
     constexpr int NK = KT / WN;            // keys of a tile that one warp sees
@@ -152,7 +157,14 @@ attn_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16
     float m_run[R2], l_run[R2];
 #pragma unroll
     for (int r = 0; r < R2; ++r) { m_run[r] = -INFINITY; l_run[r] = 0.0f; }
-    const float sl = scale * 1.4426950408889634f;           // scores in the exp2 domain
+#if SCORE_EXTRAS
+    // capped scores carry the scale already
+    const float unit = softcap > 0.0f ? 1.0f : scale;
+    const float into = softcap > 0.0f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.0f;
+#else
+    const float unit = scale;
+#endif
+    const float sl = unit * 1.4426950408889634f;            // scores in the exp2 domain
 
     load_tile(k_lo, 0);
     cp_async_commit();
@@ -189,6 +201,18 @@ attn_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16
             }
         }
 
+#if SCORE_EXTRAS
+        if (softcap > 0.0f) {        // tanh(x) = 1 - 2 / (1 + e^2x)
+#pragma unroll
+            for (int rt = 0; rt < RT; ++rt)
+#pragma unroll
+                for (int j = 0; j < NT; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+                        s[rt][j][e] = softcap - softcap * __fdividef(
+                            2.0f, 1.0f + fast_exp2(s[rt][j][e] * into));
+        }
+#endif
         // masks (only on tiles that reach a limit)
         const int key0 = kt + wn * NK;
         if (key0 + NK > min_hi || key0 < max_lo) {
@@ -295,13 +319,28 @@ attn_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16
         l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
     }
 
+    // what a row's sums are multiplied by, once its maximum m (as exponents see it) and sum l also
+    // hold the sink
+    auto with_sink = [&](int head, float& m, float& l) {
+#if SCORE_EXTRAS
+        if (sink == nullptr || (it.partial >= 0 && it.partial != it.first_partial)) return out_scale;
+        const float top = fmaxf(m, sink[head]), f = expf(m - top);       // (m -inf: f = 0)
+        l = l * f + expf(sink[head] - top);
+        m = top;
+        return f * out_scale;
+#else
+        return 1.0f;
+#endif
+    };
     if constexpr (WN == 1) {
 #pragma unroll
         for (int r = 0; r < R2; ++r) {
             if (!live[r]) continue;
             const int rt = r >> 1, i = r & 1;
+            float m = m_run[r] * unit, l = l_run[r];
+            const float f = with_sink(hq[r], m, l);
             if (it.partial < 0) {
-                const float inv = l_run[r] > 0.0f ? 1.0f / l_run[r] : 0.0f;
+                const float inv = l > 0.0f ? f / l : 0.0f;
                 __nv_bfloat16* o = out + (size_t)(tok0 + tok[r]) * out_stride + hq[r] * D;
 #pragma unroll
                 for (int j = 0; j < DT; ++j)
@@ -312,12 +351,12 @@ attn_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16
                 float* pa = partial_acc + idx * D;
 #pragma unroll
                 for (int j = 0; j < DT; ++j) {
-                    pa[j * 8 + 2 * tig] = o_acc[rt][j][2 * i];
-                    pa[j * 8 + 2 * tig + 1] = o_acc[rt][j][2 * i + 1];
+                    pa[j * 8 + 2 * tig] = o_acc[rt][j][2 * i] * f;
+                    pa[j * 8 + 2 * tig + 1] = o_acc[rt][j][2 * i + 1] * f;
                 }
                 if (tig == 0) {
-                    partial_ml[idx * 2] = m_run[r] * scale;      // natural-log domain, as merged
-                    partial_ml[idx * 2 + 1] = l_run[r];
+                    partial_ml[idx * 2] = m;                     // natural-log domain, as merged
+                    partial_ml[idx * 2 + 1] = l;
                 }
             }
         }
@@ -358,15 +397,17 @@ attn_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfloat16
                 l += red_l[w * 16 + r] * f;
                 acc += red_o[((size_t)w * 16 + r) * D + dd] * f;
             }
+            m *= unit;
+            const int t = rr / g, h = hk * g + rr % g;
+            acc *= with_sink(h, m, l);
             if (it.partial < 0) {
-                const int t = rr / g, h = hk * g + rr % g;
                 out[(size_t)(tok0 + t) * out_stride + h * D + dd] =
                     __float2bfloat16_rn(l > 0.0f ? acc / l : 0.0f);
             } else {
                 const size_t idx = ((size_t)it.partial * kv_heads + hk) * ROWS + r;
                 partial_acc[idx * D + dd] = acc;
                 if (dd == 0) {
-                    partial_ml[idx * 2] = m * scale;
+                    partial_ml[idx * 2] = m;
                     partial_ml[idx * 2 + 1] = l;
                 }
             }
@@ -381,7 +422,8 @@ int launch(const void* q, int q_stride, void* out, int out_stride, const void* k
            const void* v_pages, const int* block_table, int table_stride, int num_pages,
            const int* seq_slot, const int* seq_qstart, const int* seq_qlen, const int* seq_pos0,
            const int* items, int num_items, float* partial_acc, float* partial_ml, int heads,
-           int kv_heads, int page, float scale, int window, int* status, cudaStream_t s) {
+           int kv_heads, int page, float scale, int window, float softcap, const float* sink,
+           float out_scale, int* status, cudaStream_t s) {
     // two stages of key tiles and, unless the values are in the key pages, of value tiles
     size_t smem = (size_t)(k_pages == v_pages ? 2 : 4) * KT * LDS * sizeof(__nv_bfloat16);
     const size_t red = (size_t)WN * 16 * (D + 2) * sizeof(float);
@@ -397,7 +439,8 @@ int launch(const void* q, int q_stride, void* out, int out_stride, const void* k
                      (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)k_pages,
                      (const __nv_bfloat16*)v_pages, block_table, table_stride, num_pages, seq_slot,
                      seq_qstart, seq_qlen, seq_pos0, (const WorkItem*)items, partial_acc,
-                     partial_ml, heads, kv_heads, page, scale, window, status);
+                     partial_ml, heads, kv_heads, page, scale, window, softcap, sink, out_scale,
+                     status);
 }
 
 }  // namespace
@@ -414,8 +457,11 @@ DE_EXPORT int de_attn_mma(int shape, const void* q, int q_stride, void* out, int
                           const int* seq_qstart, const int* seq_qlen, const int* seq_pos0,
                           const int* items, int num_items, float* partial_acc, float* partial_ml,
                           int heads, int kv_heads, int head_dim, int page, float scale, int window,
-                          int* status, void* stream) {
+                          float softcap, const float* sink, float out_scale, int* status,
+                          void* stream) {
     if (num_items <= 0) return 0;
+    if (!SCORE_EXTRAS && (softcap != 0.0f || sink != nullptr || out_scale != 1.0f)) return -4;
+    if (SCORE_EXTRAS && scale <= 0.0f) return -4;        // the running maximum is of q . k
     if (head_dim != D || heads % kv_heads != 0) return -2;
     if (q_stride % 2 != 0 || out_stride % 2 != 0) return -3;
     cudaStream_t s = (cudaStream_t)stream;
@@ -423,9 +469,10 @@ DE_EXPORT int de_attn_mma(int shape, const void* q, int q_stride, void* out, int
         return launch<4, 1, WIDE_RT>(q, q_stride, out, out_stride, k_pages, v_pages, block_table,
                             table_stride, num_pages, seq_slot, seq_qstart, seq_qlen, seq_pos0, items,
                             num_items, partial_acc, partial_ml, heads, kv_heads, page, scale, window,
-                            status, s);
+                            softcap, sink, out_scale, status, s);
     return launch<1, 4, 1>(q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride,
                         num_pages, seq_slot, seq_qstart, seq_qlen, seq_pos0, items, num_items,
-                        partial_acc, partial_ml, heads, kv_heads, page, scale, window, status, s);
+                        partial_acc, partial_ml, heads, kv_heads, page, scale, window, softcap, sink,
+                        out_scale, status, s);
 }
 

@@ -15,6 +15,11 @@
 #define SPLIT_WEIGHTS 0
 #endif
 
+// 1: soft cap, sink and a factor of the results (attention_mma.cu only)
+#ifndef SCORE_EXTRAS
+#define SCORE_EXTRAS 0
+#endif
+
 namespace {
 
 constexpr int D = HEAD_DIM;

@@ -57,11 +57,17 @@ class AttentionLauncher:
 
     def __init__(self, dtype: torch.dtype, heads: int, kv_heads: int, head_dim: int,
                  scale: float, window: "int | None",
-                 device: "torch.device | None" = None, exact_weights: bool = False) -> None:
+                 device: "torch.device | None" = None, exact_weights: bool = False,
+                 extras: bool = False) -> None:
         """``exact_weights``: the softmax weights are not rounded to bfloat16 for their product
         with the values: they enter it as two bfloat16 terms (the mma.sync kernel; steps of single
-        tokens then never take the one-launch kernel)."""
+        tokens then never take the one-launch kernel).  ``extras``: the mma.sync kernel's build that
+        takes a soft cap, a sink and a factor of the results (``run``); with ``exact_weights`` and a
+        scale above 0."""
         check_head_dim(head_dim)
+        if extras and not (exact_weights and scale > 0 and uses_tensor_cores(dtype, head_dim)):
+            raise ValueError("attention: extras go with the tensor cores' exact weights and a "
+                             "scale above 0")
         if heads % kv_heads != 0:
             raise ValueError(f"heads ({heads}) must be a multiple of kv_heads ({kv_heads})")
         self.dtype, self.heads, self.kv_heads, self.head_dim = dtype, heads, kv_heads, head_dim
@@ -73,7 +79,8 @@ class AttentionLauncher:
             self.shapes = [_Shape("wide", 128 if head_dim <= 64 else 64, 0),
                            _Shape("narrow", NARROW_ROWS, 1)]
             self.module = ("attention_mma", (f"HEAD_DIM={head_dim}",)
-                           + (("SPLIT_WEIGHTS=1",) if exact_weights else ()))
+                           + (("SPLIT_WEIGHTS=1",) if exact_weights else ())
+                           + (("SCORE_EXTRAS=1",) if extras else ()))
             self.decode_module = ("attention_decode", (f"HEAD_DIM={head_dim}",))
             # prompt portions at head sizes 64 and 128: the tcgen05 kernel (tensor-memory
             # accumulators, TMA page loads) takes the wide tiles, two row tiles of 128 a block at
@@ -233,10 +240,16 @@ class AttentionLauncher:
 
     # ------------------------------------------------------------------ device side
     def run(self, q: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor,
-            v_pages: torch.Tensor, block_table: torch.Tensor, ctx) -> None:
+            v_pages: torch.Tensor, block_table: torch.Tensor, ctx, softcap: float = 0.0,
+            sink: "torch.Tensor | None" = None, out_scale: float = 1.0) -> None:
         """q: rows of [heads * d] query features at the front of each row of ``q`` (row stride
-        free); out [N, heads * d]; keys and values [pages, kv_heads, page, d]."""
+        free); out [N, heads * d]; keys and values [pages, kv_heads, page, d].  With ``extras``:
+        score <- softcap * tanh(score / softcap) where softcap is not 0; ``sink`` float32 [heads]
+        joins the softmax's denominator as exp(sink); results times ``out_scale``."""
         d = self.head_dim
+        _need(sink is None or (sink.dtype == torch.float32 and sink.is_contiguous()
+                               and sink.shape == (self.heads,)),
+              "paged attention: sink float32 [heads]")
         _need(q.stride(1) == 1 and out.stride(1) == 1 and q.dtype == out.dtype == k_pages.dtype
               == self.dtype, "paged attention: q, out and the pages must have the layer's dtype "
               "and contiguous rows")
@@ -261,7 +274,7 @@ class AttentionLauncher:
             launch_items(shape.code, module, q, out, k_pages, v_pages, block_table,
                          ctx.seq_slot, ctx.seq_qstart, ctx.seq_qlen, ctx.seq_pos0, items, combine,
                          shape.rows, acc, ml, self.heads, self.kv_heads, d, self.scale, self.window,
-                         getattr(ctx, "status", None))
+                         getattr(ctx, "status", None), (float(softcap), sink, float(out_scale)))
 
 
     def decode_step(self, ctx) -> bool:
@@ -314,8 +327,12 @@ class AttentionLauncher:
 
 def launch_items(code: int, module, q, out, k_pages, v_pages, block_table, seq_slot, seq_qstart,
                  seq_qlen, seq_pos0, items, combine, tile_rows, partial_acc, partial_ml, heads,
-                 kv_heads, head_dim, scale, window, status=None) -> None:
-    """One launch of a kernel over ``items`` and, if any range was split, the merge."""
+                 kv_heads, head_dim, scale, window, status=None,
+                 extras=(0.0, None, 1.0)) -> None:
+    """One launch of a kernel over ``items`` and, if any range was split, the merge.  ``extras``:
+    (softcap, sink, factor of the results), for the mma.sync kernel only."""
+    _need(code in (0, 1) or extras == (0.0, None, 1.0),
+          "paged attention: this kernel takes no soft cap, sink or factor")
     for name, t in (("seq_slot", seq_slot), ("seq_qstart", seq_qstart), ("seq_qlen", seq_qlen),
                     ("seq_pos0", seq_pos0), ("items", items)):
         _i32(t, name)
@@ -344,7 +361,8 @@ def launch_items(code: int, module, q, out, k_pages, v_pages, block_table, seq_s
         _check(lib.de_attn_tcgen05(*common, status.data_ptr(), _stream()),
                "paged attention (tcgen05)")
     else:
-        _check(lib.de_attn_mma(code, *common, status.data_ptr(), _stream()),
+        _check(lib.de_attn_mma(code, *common, extras[0], _ptr(extras[1]), extras[2],
+                               status.data_ptr(), _stream()),
                "paged attention (tensor cores)")
     if combine is not None and combine.shape[0] > 0:
         _i32(combine, "combine")

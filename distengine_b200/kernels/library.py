@@ -69,8 +69,8 @@ SIGNATURES: dict[str, dict[str, list]] = {
     },
     "attention_mma": {
         "de_attn_mma_head_dim": [], "de_attn_mma_rows": [I],
-        "de_attn_mma": [I, P, I, P, I, P, P, P, I, I, P, P, P, P, P, I, P, P, I, I, I, I, F, I, P,
-                        P],
+        "de_attn_mma": [I, P, I, P, I, P, P, P, I, I, P, P, P, P, P, I, P, P, I, I, I, I, F, I, F,
+                        P, F, P, P],
     },
     "attention_chunk": {
         "de_attn_chunk_rows": [I, I, I, I],
@@ -112,7 +112,7 @@ SIGNATURES: dict[str, dict[str, list]] = {
     "lru": {
         "de_lru_chunk": [], "de_lru_max_taps": [],
         "de_lru": [I, I, P, I, P, I, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, P, P, P, P, P, P, I,
-                   F, P, P, P, P],
+                   F, P, P, P, P, P],
     },
     "latent": {
         "de_latent_write": [I, I, P, I, P, I, P, I, P, P, P, F, P, F, I, I, I, I, I, P, P, I, I, I,

@@ -56,7 +56,7 @@ class Weights:
 
 def _launch(stage: int, sz: Sizes, w: Weights, x: torch.Tensor, y: torch.Tensor,
             state: torch.Tensor, out: torch.Tensor, scale: float, ctx, prod=None, local=None,
-            carry=None) -> None:
+            carry=None, terms=None) -> None:
     n, W = x.shape[0], sz.width
     for t, shape, name in ((w.x_bias, (W,), "x_bias"), (w.y_bias, (W,), "y_bias"),
                            (w.taps, (sz.taps, W), "taps"), (w.bias, (W,), "bias"),
@@ -75,6 +75,9 @@ def _launch(stage: int, sz: Sizes, w: Weights, x: torch.Tensor, y: torch.Tensor,
     for t, rows, name in ((prod, n, "prod"), (local, n, "local"), (carry, -(-n // CHUNK), "carry")):
         _need(t is None or (t.dtype == torch.float32 and t.is_contiguous()
                             and tuple(t.shape) == (rows, W)), f"lru: {name} float32 [{rows}, W]")
+    _need(terms is None or (terms.dtype == x.dtype and terms.is_contiguous()
+                            and tuple(terms.shape) == (2, n, W)),
+          "lru: terms [2, N, W] of the activation dtype")
     lib = library.load("lru")
     _check(lib.de_lru(stage, _tag(x.dtype), x.data_ptr(), x.stride(0), y.data_ptr(), y.stride(0),
                       w.x_bias.data_ptr(), w.y_bias.data_ptr(), w.taps.data_ptr(),
@@ -83,8 +86,8 @@ def _launch(stage: int, sz: Sizes, w: Weights, x: torch.Tensor, y: torch.Tensor,
                       sz.kept_offset, sz.taps, W, sz.part, n, ctx.token_seq.data_ptr(),
                       ctx.token_slot.data_ptr(), ctx.positions.data_ptr(),
                       ctx.seq_pos0.data_ptr(), ctx.seq_qlen.data_ptr(), out.data_ptr(),
-                      out.stride(0), float(scale), _ptr(prod), _ptr(local), _ptr(carry),
-                      _stream()), "lru")
+                      out.stride(0), float(scale), _ptr(terms), _ptr(prod), _ptr(local),
+                      _ptr(carry), _stream()), "lru")
 
 
 def step(sz: Sizes, w: Weights, x: torch.Tensor, y: torch.Tensor, state: torch.Tensor,
@@ -95,15 +98,16 @@ def step(sz: Sizes, w: Weights, x: torch.Tensor, y: torch.Tensor, state: torch.T
     _launch(3, sz, w, x, y, state, out, scale, ctx)
 
 
-def gates(sz, w, x, y, state, out, prod, local, ctx, scale: float = 1.0) -> None:
-    """prod and local [N, W]: S_t = prod S_start + local over the token's chunk of ``CHUNK``
+def gates(sz, w, x, y, state, out, prod, local, ctx, terms=None) -> None:
+    """``terms``: room for u's two bfloat16 terms [2, N, W], with which the gates' products go to
+    the tensor cores where the sizes allow it.  prod and local [N, W]: S_t = prod S_start + local over the token's chunk of ``CHUNK``
     consecutive tokens of the step; a sequence's first token has prod 0 and its slot's S inside."""
-    _launch(0, sz, w, x, y, state, out, scale, ctx, prod, local)
+    _launch(0, sz, w, x, y, state, out, 1.0, ctx, prod, local, terms=terms)
 
 
-def carry_on(sz, w, x, y, state, out, prod, local, carry, ctx, scale: float = 1.0) -> None:
+def carry_on(sz, w, x, y, state, out, prod, local, carry, ctx) -> None:
     """carry [chunks, W]: S at every chunk's start."""
-    _launch(1, sz, w, x, y, state, out, scale, ctx, prod, local, carry)
+    _launch(1, sz, w, x, y, state, out, 1.0, ctx, prod, local, carry)
 
 
 def finish(sz, w, x, y, state, out, prod, local, carry, ctx, scale: float = 1.0) -> None:

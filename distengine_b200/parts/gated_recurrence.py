@@ -101,7 +101,10 @@ class GatedRecurrence(ProjectedMixer):
         f32 = torch.float32
         prod = ctx.buffer("gated_recurrence.prod", (n, W), f32)
         local = ctx.buffer("gated_recurrence.local", (n, W), f32)
-        lru.gates(*common, prod, local, ctx)
+        terms = None
+        if self.dtype == torch.bfloat16:
+            terms = ctx.buffer("gated_recurrence.terms", (2, n, W))
+        lru.gates(*common, prod, local, ctx, terms)
         carry = None
         if n > lru.CHUNK:
             carry = ctx.buffer("gated_recurrence.carry", (-(-n // lru.CHUNK), W), f32)

@@ -29,7 +29,8 @@ scores.  Every one of these is a parameter:
 
 The input product stacks [q; k; v; g].  The scores, the weights and the weighted sums of the
 values are float32 (``csrc/attention_chunk.cu``); so are the convolution's sums, the norms, the
-angles and the mixing of the values.
+angles and the mixing of the values.  Without slopes and gate, bfloat16 steps go to the tensor
+cores (``csrc/attention_mma.cu``), where a weight keeps 16 bits of mantissa.
 """
 
 from __future__ import annotations
@@ -40,6 +41,7 @@ import numpy as np
 import torch
 
 from ..kernels import recurrent as rk
+from ..kernels.attention import AttentionLauncher, uses_tensor_cores
 from ..kernels.attention_plan import build_plan
 from .base import PagedKVSpec, StateSpec, compute_matrix, register_mixer
 from .context import StepPrep
@@ -119,6 +121,14 @@ class SinkAttention(ProjectedMixer):
         h = torch.arange(1, heads + 1, dtype=torch.float64)
         self.slopes = (2.0 ** (-8.0 * h / heads)).to(torch.float32).to(device) if slopes else None
         self.key = f"sink_attention/{heads // kv_heads}/{kv_heads}/{key_dim}/{value_dim}"
+        # bfloat16 without slopes and gate: the tensor cores, the softmax weights as two bfloat16
+        # terms
+        self.launcher = None
+        if (uses_tensor_cores(dtype, key_dim) and key_dim == value_dim and scale > 0
+                and not slopes and gate is None):
+            self.launcher = AttentionLauncher(dtype, heads, kv_heads, key_dim, scale, window,
+                                              device, exact_weights=True, extras=True)
+            self.key += f"/{window or 0}"            # (its work lists depend on the window)
 
     # ------------------------------------------------------------------ weights
     def _gate_rows(self) -> int:
@@ -176,7 +186,9 @@ class SinkAttention(ProjectedMixer):
         return self._host_in
 
     def kernel_modules(self):
-        return ("attention_chunk",)
+        if self.launcher is None:
+            return ("attention_chunk",)
+        return ("attention_chunk", self.launcher.module, ("attention_simt", ()))
 
     # the norms of a block that reads the stream itself never ride on this mixer's products
     def takes_unscaled(self, n_rows: int) -> bool:
@@ -204,6 +216,11 @@ class SinkAttention(ProjectedMixer):
             return
         host = prep.host
         prep.notes["sink_attention/single_tokens"] = int(host.seq_qlen.max()) == 1
+        if self.launcher is not None:
+            self.launcher.prepare(prep, allow_decode=False)
+            prep.add(name, np.zeros((0, 8), dtype=np.int32))
+            prep.notes[self.key] = -1
+            return
         if int(host.seq_qlen.max()) == 1 and rk.chunk_decode_ok(self.dtype, self.heads,
                                                                self.kv_heads, self.dk, self.dv):
             # single tokens only: the kernel that takes a (sequence, kv head) a block, no items
@@ -263,6 +280,15 @@ class SinkAttention(ProjectedMixer):
         # the gate rides in the attention kernels' last step: the heads' results are multiplied
         # in float32 and rounded once
         gate = proj[:, self.g_col: self.g_col + self._gate_rows()] if self.gate else None
+        self.attend(q, pages, gate, context, out_scale, ctx)
+
+    def attend(self, q, pages, gate, context, out_scale: float, ctx) -> None:
+        """The attention of prepared queries over the pages, gated and scaled, into ``context``."""
+        H, G, dk, dv = self.heads, self.kv_heads, self.dk, self.dv
+        if ctx.notes[self.key] == -1:
+            self.launcher.run(q, context, pages.k_pages, pages.v_pages, pages.block_table, ctx,
+                              softcap=self.softcap or 0.0, sink=self.sink, out_scale=out_scale)
+            return
         extras = dict(slopes=self.slopes, sink=self.sink, gate=gate,
                       gate_per_head=self.gate == "head", window=self.window or 0,
                       softcap=self.softcap or 0.0, out_scale=out_scale)
