@@ -241,7 +241,7 @@ __global__ void kv_write_rotated_kernel(T* __restrict__ proj, int ld, const int*
 //             a head's root mean square, so this is also the norm that follows the turn), 2 over
 //             the whole projection with weights [H dk] and [G dk]
 //   freq      the first `rot` features of every head of q and k turned by position, angle = pos *
-//             freq[i] (formed in double precision), cosine and sine times `magnitude`; pairs are
+//             freq[i] (reduced in double precision), cosine and sine times `magnitude`; pairs are
 //             (2i, 2i + 1) with `adjacent`, else (i, i + rot / 2)
 //   temp      q times 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1)
 //   mix       1: the values (as they are cached) are also left in v_first [N, G dv];
@@ -296,6 +296,15 @@ __device__ __forceinline__ void store_pair(float* p, float a, float b) {
 __device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) {
     *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
 }
+// and four
+__device__ __forceinline__ void store_four(float* p, const float4& v) {
+    *reinterpret_cast<float4*>(p) = v;
+}
+__device__ __forceinline__ void store_four(__nv_bfloat16* p, const float4& v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&a),
+                                              *reinterpret_cast<const unsigned*>(&b));
+}
 // Two sums over a block at once; every thread gets both.  The order of the additions depends on
 // the block's size only.
 __device__ __forceinline__ void block_sum2(float& a, float& b, float* scratch /* 66 floats */) {
@@ -330,7 +339,7 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, T* __rest
                                    int dk, int dv, T* __restrict__ k_pages, T* __restrict__ v_pages,
                                    const int* __restrict__ block_table, int table_stride, int page,
                                    int num_pages, int* __restrict__ status) {
-    extern __shared__ float sh[];
+    extern __shared__ __align__(16) float sh[];
     __shared__ float scratch[66];
     const int n = blockIdx.x;
     const int qk = (H + G) * dk, C = pp.v_from_k ? qk : qk + G * dv, half = pp.rot / 2;
@@ -343,10 +352,13 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, T* __rest
     const bool can_write = page_id >= 0 && page_id < num_pages;
     if (!can_write && threadIdx.x == 0) atomicExch(status, 1);   // never written outside the pool
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
-        double sn, cs;
-        sincos((double)pos * (double)pp.freq[i], &sn, &cs);
-        cs_tab[i] = (float)cs * pp.magnitude;
-        cs_tab[half + i] = (float)sn * pp.magnitude;
+        // the angle in turns, its whole turns taken off in double precision: what is left, of up to
+        // half a turn, keeps float32's digits
+        const double turns = (double)pos * ((double)pp.freq[i] * 0.15915494309189535);
+        float sn, cs;
+        sincospif((float)(2.0 * (turns - rint(turns))), &sn, &cs);
+        cs_tab[i] = cs * pp.magnitude;
+        cs_tab[half + i] = sn * pp.magnitude;
     }
     pdl_wait();
     const T* row = proj + (size_t)n * ld;
@@ -398,6 +410,12 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, T* __rest
         for (int c0 = threadIdx.x * PN; c0 < C; c0 += blockDim.x * PN) {
             float x[PN];
             load_piece(row + c0, x);
+            if (pp.bias == nullptr && pp.taps == nullptr) {      // (C is a number of pieces)
+#pragma unroll
+                for (int e = 0; e < PN; e += 4)
+                    store_four(sh + c0 + e, make_float4(x[e], x[e + 1], x[e + 2], x[e + 3]));
+                continue;
+            }
 #pragma unroll
             for (int e = 0; e < PN; ++e) {
                 x[e] += pp.bias ? pp.bias[c0 + e] : 0.0f;
@@ -424,7 +442,14 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, T* __rest
         const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
         for (int h = warp; h < H + G; h += warps) {
             float ss = 0.0f;
-            for (int i = lane; i < dk; i += 32) ss = fmaf(sh[h * dk + i], sh[h * dk + i], ss);
+            if (dk % 4 == 0) {
+                for (int i = 4 * lane; i < dk; i += 128) {
+                    const float4 v = *reinterpret_cast<const float4*>(sh + h * dk + i);
+                    ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+                }
+            } else {
+                for (int i = lane; i < dk; i += 32) ss = fmaf(sh[h * dk + i], sh[h * dk + i], ss);
+            }
             ss = warp_sum(ss);
             if (lane == 0) inv_s[h] = 1.0f / sqrtf(ss / (float)dk + pp.eps);
         }
@@ -443,69 +468,127 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ proj, int ld, T* __rest
     if (pp.temp_every > 0) temp = 1.0f + pp.temp_coef * logf((float)((pos + 1) / pp.temp_every) + 1.0f);
     const size_t at = ((size_t)(can_write ? page_id : 0) * G) * page + (size_t)(pos % page);
     const bool split = !pp.adjacent && half > 0;     // partners half a turned part apart
-    const bool paired = dk % 2 == 0 && (!split || half % 2 == 0);
-    // neighbouring features two at a time (turned together, or both plain), one store for both
-    for (int idx = threadIdx.x; idx < (paired ? (H + G) * (dk / 2) : 0); idx += blockDim.x) {
-        const int h = idx / (dk / 2), i = idx - h * (dk / 2);
-        const bool is_q = h < H;
-        if (!is_q && !can_write) continue;
-        const float* x = sh + h * dk;
-        const float* wt = nullptr;
-        float inv = 1.0f;
-        if (pp.norm != 0) {
-            inv = inv_s[h];
-            wt = is_q ? pp.q_weight : pp.k_weight;
-            if (pp.norm == 2) wt += (is_q ? h : h - H) * dk;
-        }
-        const float mul = is_q ? temp : 1.0f;
-        T* dst = is_q ? q_out + (size_t)n * (H * dk) + h * dk
-                      : k_pages + (at + (size_t)(h - H) * page) * dk;
-        const int a = 2 * i, b = a + 1;
-        float ra = x[a] * inv * (wt ? wt[a] : 1.0f), rb = x[b] * inv * (wt ? wt[b] : 1.0f);
-        if (split && a < pp.rot) {                   // both features lie in one half of the turned part
-            const bool first = a < half;
-            const int p = first ? a : a - half, o = first ? a + half : a - half;
-            const float oa = x[o] * inv * (wt ? wt[o] : 1.0f);
-            const float ob = x[o + 1] * inv * (wt ? wt[o + 1] : 1.0f);
-            float other;
-            if (first) {
-                rope_rotate(ra, oa, cs_tab[p], cs_tab[half + p], ra, other);
-                rope_rotate(rb, ob, cs_tab[p + 1], cs_tab[half + p + 1], rb, other);
-            } else {
-                rope_rotate(oa, ra, cs_tab[p], cs_tab[half + p], other, ra);
-                rope_rotate(ob, rb, cs_tab[p + 1], cs_tab[half + p + 1], other, rb);
+    if (dk % 4 == 0 && dv % 4 == 0 && pp.rot % (split ? 8 : 4) == 0 && C % 4 == 0) {
+        // a warp a head, four neighbouring features a lane (turned together, or all plain)
+        const int lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+        auto four = [](const float* p) { return *reinterpret_cast<const float4*>(p); };
+        for (int h = threadIdx.x >> 5; h < H + G; h += warps) {
+            const bool is_q = h < H;
+            if (!is_q && !can_write) continue;
+            const float* x = sh + h * dk;
+            const float* wt = pp.norm == 0 ? nullptr : is_q ? pp.q_weight : pp.k_weight;
+            if (wt && pp.norm == 2) wt += (is_q ? h : h - H) * dk;
+            const float inv = pp.norm != 0 ? inv_s[h] : 1.0f, mul = is_q ? temp : 1.0f;
+            T* dst = is_q ? q_out + (size_t)n * (H * dk) + h * dk
+                          : k_pages + (at + (size_t)(h - H) * page) * dk;
+            auto normed = [&](int i) {
+                float4 v = four(x + i);
+                v.x *= inv; v.y *= inv; v.z *= inv; v.w *= inv;
+                if (wt) {
+                    const float w0 = wt[i], w1 = wt[i + 1], w2 = wt[i + 2], w3 = wt[i + 3];
+                    v.x *= w0; v.y *= w1; v.z *= w2; v.w *= w3;
+                }
+                return v;
+            };
+            for (int i = 4 * lane; i < dk; i += 128) {
+                float4 v = normed(i);
+                float other;
+                if (split && i < pp.rot) {
+                    const bool first = i < half;
+                    const int p = first ? i : i - half;
+                    const float4 o = normed(first ? i + half : i - half);
+                    const float4 c = four(cs_tab + p), s = four(cs_tab + half + p);
+                    if (first) {
+                        rope_rotate(v.x, o.x, c.x, s.x, v.x, other);
+                        rope_rotate(v.y, o.y, c.y, s.y, v.y, other);
+                        rope_rotate(v.z, o.z, c.z, s.z, v.z, other);
+                        rope_rotate(v.w, o.w, c.w, s.w, v.w, other);
+                    } else {
+                        rope_rotate(o.x, v.x, c.x, s.x, other, v.x);
+                        rope_rotate(o.y, v.y, c.y, s.y, other, v.y);
+                        rope_rotate(o.z, v.z, c.z, s.z, other, v.z);
+                        rope_rotate(o.w, v.w, c.w, s.w, other, v.w);
+                    }
+                } else if (!split && i < pp.rot) {
+                    const float* c = cs_tab + i / 2;
+                    rope_rotate(v.x, v.y, c[0], c[half], v.x, v.y);
+                    rope_rotate(v.z, v.w, c[1], c[half + 1], v.z, v.w);
+                }
+                v.x *= mul; v.y *= mul; v.z *= mul; v.w *= mul;
+                store_four(dst + i, v);
             }
-        } else if (!split && i < half) {
-            rope_rotate(ra, rb, cs_tab[i], cs_tab[half + i], ra, rb);
         }
-        store_pair(dst + a, ra * mul, rb * mul);
-    }
-    const int per = dk - half;                       // work items a head: pairs, then plain features
-    for (int idx = threadIdx.x; idx < (paired ? 0 : (H + G) * per); idx += blockDim.x) {
-        const int h = idx / per, i = idx - h * per;
-        const bool is_q = h < H;
-        if (!is_q && !can_write) continue;
-        const float* x = sh + h * dk;
-        const float* wt = nullptr;
-        float inv = 1.0f;
-        if (pp.norm != 0) {
-            inv = inv_s[h];
-            wt = is_q ? pp.q_weight : pp.k_weight;
-            if (pp.norm == 2) wt += (is_q ? h : h - H) * dk;
+        if (pp.mix == 0) {
+            for (int h = threadIdx.x >> 5; h < (can_write ? G : 0); h += warps)
+                for (int i = 4 * lane; i < dv; i += 128)
+                    store_four(v_pages + (at + (size_t)h * page) * dv + i, four(sh + v_col + h * dv + i));
+            return;
         }
-        const float mul = is_q ? temp : 1.0f;
-        T* dst = is_q ? q_out + (size_t)n * (H * dk) + h * dk
-                      : k_pages + (at + (size_t)(h - H) * page) * dk;
-        if (i < half) {
-            const int a = pp.adjacent ? 2 * i : i, b = pp.adjacent ? 2 * i + 1 : i + half;
-            float ra, rb;
-            rope_rotate(x[a] * inv * (wt ? wt[a] : 1.0f), x[b] * inv * (wt ? wt[b] : 1.0f),
-                        cs_tab[i], cs_tab[half + i], ra, rb);
-            dst[a] = from_float<T>(ra * mul);
-            dst[b] = from_float<T>(rb * mul);
-        } else {
-            const int a = i + half;
-            dst[a] = from_float<T>(x[a] * inv * (wt ? wt[a] : 1.0f) * mul);
+    } else {
+        const bool paired = dk % 2 == 0 && (!split || half % 2 == 0);
+        // neighbouring features two at a time (turned together, or both plain), one store for both
+        for (int idx = threadIdx.x; idx < (paired ? (H + G) * (dk / 2) : 0); idx += blockDim.x) {
+            const int h = idx / (dk / 2), i = idx - h * (dk / 2);
+            const bool is_q = h < H;
+            if (!is_q && !can_write) continue;
+            const float* x = sh + h * dk;
+            const float* wt = nullptr;
+            float inv = 1.0f;
+            if (pp.norm != 0) {
+                inv = inv_s[h];
+                wt = is_q ? pp.q_weight : pp.k_weight;
+                if (pp.norm == 2) wt += (is_q ? h : h - H) * dk;
+            }
+            const float mul = is_q ? temp : 1.0f;
+            T* dst = is_q ? q_out + (size_t)n * (H * dk) + h * dk
+                          : k_pages + (at + (size_t)(h - H) * page) * dk;
+            const int a = 2 * i, b = a + 1;
+            float ra = x[a] * inv * (wt ? wt[a] : 1.0f), rb = x[b] * inv * (wt ? wt[b] : 1.0f);
+            if (split && a < pp.rot) {                   // both features lie in one half of the turned part
+                const bool first = a < half;
+                const int p = first ? a : a - half, o = first ? a + half : a - half;
+                const float oa = x[o] * inv * (wt ? wt[o] : 1.0f);
+                const float ob = x[o + 1] * inv * (wt ? wt[o + 1] : 1.0f);
+                float other;
+                if (first) {
+                    rope_rotate(ra, oa, cs_tab[p], cs_tab[half + p], ra, other);
+                    rope_rotate(rb, ob, cs_tab[p + 1], cs_tab[half + p + 1], rb, other);
+                } else {
+                    rope_rotate(oa, ra, cs_tab[p], cs_tab[half + p], other, ra);
+                    rope_rotate(ob, rb, cs_tab[p + 1], cs_tab[half + p + 1], other, rb);
+                }
+            } else if (!split && i < half) {
+                rope_rotate(ra, rb, cs_tab[i], cs_tab[half + i], ra, rb);
+            }
+            store_pair(dst + a, ra * mul, rb * mul);
+        }
+        const int per = dk - half;                       // work items a head: pairs, then plain features
+        for (int idx = threadIdx.x; idx < (paired ? 0 : (H + G) * per); idx += blockDim.x) {
+            const int h = idx / per, i = idx - h * per;
+            const bool is_q = h < H;
+            if (!is_q && !can_write) continue;
+            const float* x = sh + h * dk;
+            const float* wt = nullptr;
+            float inv = 1.0f;
+            if (pp.norm != 0) {
+                inv = inv_s[h];
+                wt = is_q ? pp.q_weight : pp.k_weight;
+                if (pp.norm == 2) wt += (is_q ? h : h - H) * dk;
+            }
+            const float mul = is_q ? temp : 1.0f;
+            T* dst = is_q ? q_out + (size_t)n * (H * dk) + h * dk
+                          : k_pages + (at + (size_t)(h - H) * page) * dk;
+            if (i < half) {
+                const int a = pp.adjacent ? 2 * i : i, b = pp.adjacent ? 2 * i + 1 : i + half;
+                float ra, rb;
+                rope_rotate(x[a] * inv * (wt ? wt[a] : 1.0f), x[b] * inv * (wt ? wt[b] : 1.0f),
+                            cs_tab[i], cs_tab[half + i], ra, rb);
+                dst[a] = from_float<T>(ra * mul);
+                dst[b] = from_float<T>(rb * mul);
+            } else {
+                const int a = i + half;
+                dst[a] = from_float<T>(x[a] * inv * (wt ? wt[a] : 1.0f) * mul);
+            }
         }
     }
     if (pp.mix == 0 && dv % 2 == 0) {                // plain values, two at a time

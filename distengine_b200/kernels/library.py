@@ -160,6 +160,8 @@ def default_build_requests() -> list[tuple[str, tuple[str, ...]]]:
     # (16 and 32: what the tiny models that the smoke test generates with have)
     return (requests + [("attention_mma", (f"HEAD_DIM={d}",)) for d in (16, 64, 128)]
             + [("attention_mma", ("HEAD_DIM=32", "SPLIT_WEIGHTS=1"))]
+            + [("attention_mma", (f"HEAD_DIM={d}", "SPLIT_WEIGHTS=1", "SCORE_EXTRAS=1"))
+               for d in (16, 32, 64, 128)]
             + [("attention_tcgen05", (f"HEAD_DIM={d}",)) for d in (64, 128)]
             + [("attention_decode", (f"HEAD_DIM={d}",)) for d in (16, 64, 128)])
 
