@@ -84,6 +84,7 @@ ATTENTIONS = [
     (sc.attention(12, 1, 8, 0.3, None, (1000000.0, 4)), 16),
     (sc.attention(5, 5, 24, 0.3, 1), 8),
     (sc.attention(4, 4, 128, 0.1, 33, (500.0, 128, 2.0), 3.0), 32),
+    (sc.attention(6, 3, 80, 0.12, 40, (500.0, 40)), 16),
 ]
 
 
