@@ -193,7 +193,8 @@ attn_combine_kernel(T* __restrict__ out, int out_stride, const int* __restrict__
     const int g = heads / kv_heads;
     const int rows_total = seq_qlen[it.seq] * g;
     const int lane = threadIdx.x & 31;
-    for (int w = threadIdx.x >> 5; w < rows_per_tile; w += ROWS) {
+    // a warp a row, the rows of a tile over blockIdx.z
+    for (int w = blockIdx.z * ROWS + (threadIdx.x >> 5); w < rows_per_tile; w += ROWS * gridDim.z) {
         const int r = it.row0 + w;
         if (r >= rows_total) continue;
         const int t = r / g, hq = hk * g + r % g;
@@ -206,17 +207,20 @@ attn_combine_kernel(T* __restrict__ out, int out_stride, const int* __restrict__
         float acc[MAX_D / 32];
 #pragma unroll
         for (int i = 0; i < MAX_D / 32; ++i) acc[i] = 0.0f;
+        // (everything is loaded without a branch on what was loaded before it)
+#pragma unroll 4
         for (int c = 0; c < it.num_partials; ++c) {
             const size_t idx = ((size_t)(it.first_partial + c) * kv_heads + hk) * rows_per_tile + w;
-            const float mc = partial_ml[idx * 2];
-            if (mc == -INFINITY) continue;            // the chunk held no visible key
-            const float f = expf(mc - m);
-            l += partial_ml[idx * 2 + 1] * f;
+            const float mc = partial_ml[idx * 2], lc = partial_ml[idx * 2 + 1];
+            const bool any = mc != -INFINITY;         // else the chunk held no visible key
+            const float f = any ? expf(mc - m) : 0.0f;
+            if (any) l += lc * f;
             const float* pa = partial_acc + idx * d;
 #pragma unroll
             for (int i = 0; i < MAX_D / 32; ++i) {
                 const int dd = lane + 32 * i;
-                if (dd < d) acc[i] = fmaf(pa[dd], f, acc[i]);
+                const float v = dd < d ? pa[dd] : 0.0f;
+                if (any) acc[i] = fmaf(v, f, acc[i]);
             }
         }
         const float inv = l > 0.0f ? 1.0f / l : 0.0f;
@@ -309,7 +313,7 @@ static int launch_combine(int dtype, void* out, int out_stride, const int* seq_q
     if (num_items <= 0) return 0;
     if (d <= 0 || d > MAX_D) return -2;
     cudaStream_t s = (cudaStream_t)stream;
-    dim3 grid(num_items, kv_heads);
+    dim3 grid(num_items, kv_heads, (rows_per_tile + ROWS - 1) / ROWS);
     if (dtype == DE_BF16)
         return de_launch(attn_combine_kernel<__nv_bfloat16>, grid, dim3(ROWS * 32), 0, s,
                          (__nv_bfloat16*)out, out_stride, seq_qstart, seq_qlen,
